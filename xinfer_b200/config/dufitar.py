@@ -25,30 +25,11 @@ from typing import Any, Mapping, Optional, Tuple
 from .errors import ConfigError
 from .plan import (AttentionSpec, BlockOp, BlockSpec, DynamicTanhSpec, FeedForwardSpec, LatentAttentionSpec, LayerRun,
                    ModelPlan, RopeSpec, YarnScaling)
+from .reading import integer as _int, need as _get, number as _num
 
 ARCHITECTURE = "Dufitar"
 # the engine's own bound on a sequence: this design has no position table and names no limit
 MAX_POSITIONS = 1 << 20
-
-
-def _get(raw, key: str, where: str):
-    if not isinstance(raw, Mapping) or key not in raw or raw[key] is None:
-        raise ConfigError(f"config.json lacks '{where}{key}'")
-    return raw[key]
-
-
-def _int(raw, key: str, where: str, least: int = 1) -> int:
-    v = _get(raw, key, where)
-    if isinstance(v, bool) or not isinstance(v, int) or v < least:
-        raise ConfigError(f"config key '{where}{key}' must be an integer >= {least}, got {v!r}")
-    return v
-
-
-def _num(raw, key: str, where: str, positive: bool = False) -> float:
-    v = _get(raw, key, where)
-    if isinstance(v, bool) or not isinstance(v, (int, float)) or (positive and not v > 0):
-        raise ConfigError(f"config key '{where}{key}' must be a{' positive' if positive else ''} number, got {v!r}")
-    return float(v)
 
 
 @dataclass(frozen=True)

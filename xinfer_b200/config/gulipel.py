@@ -28,31 +28,12 @@ from typing import Any, Mapping, Optional, Tuple
 from .errors import ConfigError
 from .plan import (AttentionSpec, BlockOp, BlockSpec, FeedForwardSpec, GatedDeltaSpec, LayerRun, ModelPlan, NormSpec,
                    PairEmbeddingSpec, ParallelMixerSpec, SelectiveStateSpec, TokenSideSpec)
+from .reading import integer as _int, need as _get, number as _num
 
 ARCHITECTURE = "Gulipel"
 # the engine's own bound on a sequence where the model has no position table
 MAX_POSITIONS = 1 << 20
 STATE_SPACE_TYPES = ("mamba2", "mamba2_2")
-
-
-def _get(raw, key: str, where: str):
-    if not isinstance(raw, Mapping) or key not in raw or raw[key] is None:
-        raise ConfigError(f"config.json lacks '{where}{key}'")
-    return raw[key]
-
-
-def _int(raw, key: str, where: str, least: int = 1) -> int:
-    v = _get(raw, key, where)
-    if isinstance(v, bool) or not isinstance(v, int) or v < least:
-        raise ConfigError(f"config key '{where}{key}' must be an integer >= {least}, got {v!r}")
-    return v
-
-
-def _num(raw, key: str, where: str, positive: bool = False) -> float:
-    v = _get(raw, key, where)
-    if isinstance(v, bool) or not isinstance(v, (int, float)) or (positive and not v > 0):
-        raise ConfigError(f"config key '{where}{key}' must be a{' positive' if positive else ''} number, got {v!r}")
-    return float(v)
 
 
 def _opt_int(raw, key: str, where: str) -> Optional[int]:

@@ -170,9 +170,13 @@ class LatentAttentionSpec(PartSpec):
     ``rope_dim`` rotated query channels; its plain key is ``W_uk,h c`` and its value ``W_uv,h c`` (``v_head_dim``
     channels).  ``window`` as for attention.  ``sink``: every head's softmax has one more entry with a learned score
     and no value.  ``gate``: the concatenated heads are multiplied by ``sigmoid(W_g h)`` before the output projection.
-    ``shares_cache``: the layer has no latent projection of its own and reads the rows another layer cached.
+    ``gate_per_head``: the gate is one number per head (W_g has ``num_heads`` rows) instead of one per channel.
+    ``shares_cache``: the layer has no latent projection of its own and reads the rows another layer cached;
+    ``row_tail`` of their last channels (the owner's rotated key part) are not this layer's and take no part.
     ``cache_window``: how long cached rows must be kept (None: for ever): the largest window among the layers that
-    read them.  ``names``: the tensors q, latent projection, its norm, uk, uv, sink, gate, output after the prefix."""
+    read them.  ``rope_dim`` 0 (and ``rope`` None): no positions.  ``q_rank``: the queries go through a latent of
+    their own, ``W_uq (W_dq h / rms * w)`` (``norm_eps``), instead of one matrix.  ``names``: the tensors q, latent
+    projection, its norm, uk, uv, sink, gate, output after the prefix; ``q_names``: W_dq, its norm, W_uq."""
 
     hidden: int = 0
     num_heads: int = 0
@@ -189,6 +193,10 @@ class LatentAttentionSpec(PartSpec):
     gate: bool = False
     shares_cache: bool = False
     names: Tuple[str, ...] = ("q", "dkv", "dkv.norm", "uk", "uv", "sink", "g", "o")
+    gate_per_head: bool = False
+    row_tail: int = 0
+    q_rank: Optional[int] = None
+    q_names: Tuple[str, ...] = ("dq", "dq.norm", "uq")
 
 
 @dataclass(frozen=True)
@@ -249,6 +257,40 @@ class GatedDeltaSpec(PartSpec):
 
 
 @dataclass(frozen=True)
+class GatedLinearAttentionSpec(PartSpec):
+    """Linear attention that forgets per key channel: q and k of ``heads x head_dim``, v of ``heads x v_head_dim``, a
+    decay per (head, key channel) alpha = sigmoid(W_a2 (W_a1 h) + b)^(1 / tau); per head S <- diag(alpha) S + k v^T,
+    o = S^T q head_dim^-1/2 (read after the token's own write); o is RMS-normed per head (``eps``) with one weight
+    shared by the heads, multiplied by silu(W_g h), then projected out.  ``decay_rank``: the inner size of the
+    low-rank map; None: whatever the tensors' shapes say (the random-weights mode then draws ``DEFAULT_RANK``).
+    ``names``: q, k, v, W_g, output, norm, W_a1, W_a2, b after the prefix."""
+
+    hidden: int = 0
+    heads: int = 0
+    head_dim: int = 0
+    v_head_dim: int = 0
+    tau: float = 1.0
+    eps: float = 1e-6
+    decay_rank: Optional[int] = None
+    names: Tuple[str, ...] = ("q", "k", "v", "g", "o", "norm", "a1", "a2", "a2.b")
+
+    DEFAULT_RANK = 16
+
+
+@dataclass(frozen=True)
+class InputConvSpec(PartSpec):
+    """A mixer whose input is first replaced by ``h + conv(h)``, a causal convolution of ``taps`` taps per channel
+    (no bias, no activation) whose last ``taps - 1`` inputs are carried per request.  ``name``: the filter's tensor
+    ``[hidden, taps]``; ``inner_name``: the name piece of the mixer's own tensors, both after the prefix."""
+
+    hidden: int = 0
+    inner: Optional[PartSpec] = None
+    taps: int = 1
+    name: str = "conv"
+    inner_name: str = ""
+
+
+@dataclass(frozen=True)
 class ParallelMixerSpec(PartSpec):
     """Two mixers that read the same input; the result is left_scale * left + right_scale * right.
     ``out_norms`` = (left name, right name): each mixer's result (after its own output projection) is first
@@ -282,12 +324,15 @@ class FeedForwardSpec(PartSpec):
 @dataclass(frozen=True)
 class RoutedExpertsSpec(PartSpec):
     """``experts`` small gated feed-forwards (``e0.``, ``e1.``, ... after the prefix, without biases) of which a
-    learned router gives every token ``top``.  Scores are ``sigmoid(W_router h)`` in float32; the choice is made
+    learned router gives every token ``top``.  Scores are ``sigmoid(W_router h)`` (``score`` "softmax": the softmax
+    over all experts) in float32; the choice is made
     on ``score + correction`` (a learned vector; ``correction`` False: on the scores), the weights are the chosen
-    experts' plain scores (``renormalize``: divided by their sum).  Experts form ``groups`` equal groups of
+    experts' plain scores (``renormalize``: divided by their sum plus ``renormalize_eps``) times ``weight_scale``.
+    Experts form ``groups`` equal groups of
     neighbours; a group's score is the sum of its ``group_best`` largest choice scores and only experts of the
     ``keep`` best groups can be chosen.  ``activation`` / ``act_params`` as in ``FeedForwardSpec``.  ``shared``:
-    a gated feed-forward of its own sizes (``shared.`` after the prefix) that every token runs and that is added."""
+    a gated feed-forward of its own sizes (``shared.`` after the prefix) that every token runs and that is added,
+    with ``shared_gate`` (a tensor name after the prefix) times the sigmoid of one number per token."""
 
     hidden: int = 0
     intermediate: int = 0
@@ -301,6 +346,10 @@ class RoutedExpertsSpec(PartSpec):
     activation: str = "silu"
     act_params: Tuple[float, ...] = ()
     shared: Optional[FeedForwardSpec] = None
+    score: str = "sigmoid"
+    renormalize_eps: float = 0.0
+    weight_scale: float = 1.0
+    shared_gate: Optional[str] = None
 
 
 @dataclass(frozen=True)

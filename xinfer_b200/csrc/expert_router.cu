@@ -1,12 +1,14 @@
 // A learned router over experts with a per-expert score and a choice among groups of experts.
+// `w_r` holds a row per expert and, where a gate is asked for, one more.
 //
 //   z_e      = W_r[e, :] . h                      float32 (h may arrive in the engine's type)
-//   s_e      = sigmoid(z_e)                       the score, also the chosen expert's weight
+//   s_e      = sigmoid(z_e), or softmax(z)_e over all experts       the score, also the chosen expert's weight
 //   c_e      = s_e + correction_e                 the choice score (correction absent: c = s)
 //   group g  = experts g * E/groups .. (g + 1) * E/groups - 1; its score: the sum of its `group_best` largest c
 //   allowed  = the experts of the `keep` groups with the largest scores (the others count as minus infinity)
 //   chosen   = the `top` allowed experts with the largest c; weight of a chosen expert: s_e (not renormalized),
-//              or s_e / sum of the chosen s where `renorm` is set
+//              or s_e / (sum of the chosen s + renorm_eps) where `renorm` is set; times `weight_scale`
+//   gate     = sigmoid(w_g . h), one number per token (a further row of the matrix; absent: none)
 //
 // One block of four warps takes ROUTER_TOKENS consecutive tokens: one, so that a step of few tokens still spreads over
 // the machine (blocks that run on one SM at the same time find the matrix in its L1), or two for steps of thousands
@@ -39,18 +41,20 @@ template <typename T, int ROUTER_TOKENS>
 __global__ void __launch_bounds__(ROUTER_THREADS)
 expert_router_kernel(int* __restrict__ choice, float* __restrict__ weight, const T* __restrict__ h,
                      const float* __restrict__ w_r, const float* __restrict__ correction,
-                     const int* __restrict__ req_of_token, int tokens, int E, int K, int top, int groups, int keep,
-                     int group_best, int renorm, int vec4) {
+                     const int* __restrict__ req_of_token, float* __restrict__ gate, int tokens, int E, int K, int top,
+                     int groups, int keep, int group_best, int softmax, int renorm, float renorm_eps, float weight_scale,
+                     int vec4) {
     extern __shared__ float sm[];
-    float* s_all = sm;                                   // [tokens of the block][E] logits, then scores
-    float* c_all = sm + ROUTER_TOKENS * E;               // [..][E] choice scores (minus infinity once taken or not allowed)
-    float* g_all = sm + 2 * ROUTER_TOKENS * E;           // [..][groups]
+    const int rows = E + (gate != nullptr ? 1 : 0);      // rows of the matrix: the experts, then the gate's
+    float* s_all = sm;                                   // [tokens of the block][rows] logits, then scores
+    float* c_all = sm + ROUTER_TOKENS * rows;            // [..][rows] choice scores (minus infinity once taken or not allowed)
+    float* g_all = sm + 2 * ROUTER_TOKENS * rows;        // [..][groups]
     const int t0 = blockIdx.x * ROUTER_TOKENS, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarps = blockDim.x >> 5;
     const int nt = min(ROUTER_TOKENS, tokens - t0);
     // a warp takes two experts at a time (e and e + nwarps): twice the loads in flight for the same chain of sums
-    for (int e = warp; e < E; e += 2 * nwarps) {
+    for (int e = warp; e < rows; e += 2 * nwarps) {
         const int e2 = e + nwarps;
-        const bool two = e2 < E;
+        const bool two = e2 < rows;
         const float* wa = w_r + (size_t)e * K;
         const float* wb = w_r + (size_t)(two ? e2 : e) * K;
         float acc[ROUTER_TOKENS], acc2[ROUTER_TOKENS];
@@ -93,8 +97,8 @@ expert_router_kernel(int* __restrict__ choice, float* __restrict__ weight, const
         for (int j = 0; j < ROUTER_TOKENS; ++j) {
             const float z = warp_sum(acc[j]), z2 = warp_sum(acc2[j]);
             if (lane == 0) {
-                s_all[j * E + e] = z;
-                if (two) s_all[j * E + e2] = z2;
+                s_all[j * rows + e] = z;
+                if (two) s_all[j * rows + e2] = z2;
             }
         }
     }
@@ -102,9 +106,10 @@ expert_router_kernel(int* __restrict__ choice, float* __restrict__ weight, const
     const int per = E / groups;
     for (int j = warp; j < nt; j += nwarps) {
         const int t = t0 + j;
-        float* s = s_all + j * E;
-        float* c = c_all + j * E;
+        float* s = s_all + j * rows;
+        float* c = c_all + j * rows;
         float* gs = g_all + j * groups;
+        if (gate != nullptr && lane == 0) gate[t] = req_of_token[t] < 0 ? 0.f : 1.f / (1.f + expf(-s[E]));
         if (req_of_token[t] < 0) {
             for (int k = lane; k < top; k += 32) {
                 choice[(size_t)t * top + k] = 0;
@@ -112,8 +117,16 @@ expert_router_kernel(int* __restrict__ choice, float* __restrict__ weight, const
             }
             continue;
         }
+        float top_z = -CUDART_INF_F, inv_sum = 1.f;
+        if (softmax) {
+            for (int e = lane; e < E; e += 32) top_z = fmaxf(top_z, s[e]);
+            top_z = warp_max(top_z);
+            float sum = 0.f;
+            for (int e = lane; e < E; e += 32) sum += expf(s[e] - top_z);
+            inv_sum = 1.f / warp_sum(sum);
+        }
         for (int e = lane; e < E; e += 32) {
-            const float v = 1.f / (1.f + expf(-s[e]));
+            const float v = softmax ? expf(s[e] - top_z) * inv_sum : 1.f / (1.f + expf(-s[e]));
             s[e] = v;
             c[e] = v + (correction != nullptr ? correction[e] : 0.f);
         }
@@ -178,28 +191,32 @@ expert_router_kernel(int* __restrict__ choice, float* __restrict__ weight, const
             }
             __syncwarp();
         }
-        if (renorm && total > 0.f)
-            for (int k = lane; k < top; k += 32) weight[(size_t)t * top + k] /= total;
+        if ((renorm && total > 0.f) || weight_scale != 1.f) {
+            const float div = renorm && total > 0.f ? total + renorm_eps : 1.f;
+            for (int k = lane; k < top; k += 32) weight[(size_t)t * top + k] = weight[(size_t)t * top + k] / div * weight_scale;
+        }
     }
 }
 
 XB_EXPORT int xb_expert_router(int dtype, int* choice, float* weight, const void* h, const float* w_r, const float* correction,
-                               const int* req_of_token, int tokens, int experts, int K, int top, int groups, int keep,
-                               int group_best, int renorm, cudaStream_t stream) {
+                               const int* req_of_token, float* gate, int tokens, int experts, int K, int top, int groups,
+                               int keep, int group_best, int softmax, int renorm, float renorm_eps, float weight_scale,
+                               cudaStream_t stream) {
     if (tokens <= 0) return 0;
     if (experts <= 0 || top <= 0 || top > experts || groups <= 0 || experts % groups || keep <= 0 || keep > groups ||
         group_best <= 0 || group_best > 8)
         return (int)cudaErrorInvalidValue;
     const int per_block = tokens >= 4096 ? 2 : 1;
-    const size_t smem = (size_t)per_block * (2 * (size_t)experts + groups) * sizeof(float);
+    const size_t smem = (size_t)per_block * (2 * ((size_t)experts + 1) + groups) * sizeof(float);
     if (smem > 48 * 1024) return (int)cudaErrorInvalidValue;
     const size_t esz = dtype == XB_F32 ? 4 : 2;
     const int vec4 = (K % 4 == 0 && !((uintptr_t)h & (4 * esz - 1)) && !((uintptr_t)w_r & 15)) ? 1 : 0;
     const unsigned blocks = (unsigned)((tokens + per_block - 1) / per_block);
 #define XB_ROUTER(T, N)                                                                                                   \
     expert_router_kernel<T, N><<<blocks, ROUTER_THREADS, smem, stream>>>(choice, weight, (const T*)h, w_r, correction,    \
-                                                                         req_of_token, tokens, experts, K, top, groups,   \
-                                                                         keep, group_best, renorm, vec4)
+                                                                         req_of_token, gate, tokens, experts, K, top,     \
+                                                                         groups, keep, group_best, softmax, renorm,       \
+                                                                         renorm_eps, weight_scale, vec4)
     if (dtype == XB_F32) {
         if (per_block == 2) XB_ROUTER(float, 2); else XB_ROUTER(float, 1);
     } else {

@@ -210,13 +210,24 @@ XB_EXPORT int xb_expert_gemm(int in_dtype, int out_dtype, void* y, const void* a
 // so that ONE product with the down matrices side by side along K sums the token's experts.
 // ------------------------------------------------------------------------------------------
 // `weights` [T, top] (absent: every chosen expert weighs 1 / top); no ids: the table has a row per token.
+// Behind the experts a row may hold one more gated feed-forward, F_dense wide, that every token runs, with a weight per
+// token (dense_weight):  act[t, E * F + f] = dense_weight[t] * act(gu[t, E*2F + f], gu[t, E*2F + F_dense + f]).
 template <typename T>
 __global__ void expert_select_gate_kernel(T* __restrict__ act, const T* __restrict__ gu, const int* __restrict__ table,
                                           const int* __restrict__ ids, const int* __restrict__ sampled, int num_sampled,
-                                          const int* __restrict__ req_of_token, int top, int E, int F, int vocab,
-                                          float weight, const float* __restrict__ weights, int code, float p0, float p1,
-                                          int* err) {
+                                          const int* __restrict__ req_of_token, int top, int E, int F, int F_dense, int vocab,
+                                          float weight, const float* __restrict__ weights,
+                                          const float* __restrict__ dense_weight, int code, float p0, float p1, int* err) {
     const int t = blockIdx.x, e = blockIdx.y;
+    const T* gu_row = gu + (size_t)t * 2 * ((size_t)E * F + F_dense);
+    T* act_row = act + (size_t)t * ((size_t)E * F + F_dense);
+    if (e == E) {
+        const T* g = gu_row + (size_t)E * 2 * F;
+        const float dw = dense_weight[t];
+        for (int f = threadIdx.x; f < F_dense; f += blockDim.x)
+            act_row[(size_t)E * F + f] = from_f32<T>(gate_mul_any(code, to_f32<T>(g[f]), to_f32<T>(g[F_dense + f]), p0, p1) * dw);
+        return;
+    }
     int id = ids != nullptr ? ids[t] : t;
     if (id < 0 && sampled != nullptr && -1 - id < num_sampled) id = sampled[-1 - id];
     bool chosen = false;
@@ -231,8 +242,8 @@ __global__ void expert_select_gate_kernel(T* __restrict__ act, const T* __restri
                 }
         }
     }
-    const T* g = gu + ((size_t)t * E + e) * 2 * F;
-    T* o = act + ((size_t)t * E + e) * F;
+    const T* g = gu_row + (size_t)e * 2 * F;
+    T* o = act_row + (size_t)e * F;
     for (int f = threadIdx.x; f < F; f += blockDim.x) {
         float v = 0.f;
         if (chosen) v = gate_mul_any(code, to_f32<T>(g[f]), to_f32<T>(g[F + f]), p0, p1) * weight;
@@ -241,19 +252,22 @@ __global__ void expert_select_gate_kernel(T* __restrict__ act, const T* __restri
 }
 
 XB_EXPORT int xb_expert_select_gate(int dtype, void* act, const void* gu, const int* table, const int* ids, const int* sampled,
-                                    int num_sampled, const int* req_of_token, int tokens, int top, int experts, int F, int vocab,
-                                    const float* weights, int code, float p0, float p1, int* err, cudaStream_t stream) {
+                                    int num_sampled, const int* req_of_token, int tokens, int top, int experts, int F,
+                                    int F_dense, int vocab, const float* weights, const float* dense_weight, int code, float p0,
+                                    float p1, int* err, cudaStream_t stream) {
     if (tokens <= 0) return 0;
-    const dim3 grid(tokens, experts);
+    if (F_dense > 0 && dense_weight == nullptr) return (int)cudaErrorInvalidValue;
+    const dim3 grid(tokens, experts + (F_dense > 0 ? 1 : 0));
     const float weight = 1.f / (float)top;
     if (dtype == XB_F32)
         expert_select_gate_kernel<float><<<grid, 256, 0, stream>>>((float*)act, (const float*)gu, table, ids, sampled, num_sampled,
-                                                                   req_of_token, top, experts, F, vocab, weight, weights, code,
-                                                                   p0, p1, err);
+                                                                   req_of_token, top, experts, F, F_dense, vocab, weight,
+                                                                   weights, dense_weight, code, p0, p1, err);
     else
         expert_select_gate_kernel<__nv_bfloat16><<<grid, 256, 0, stream>>>((__nv_bfloat16*)act, (const __nv_bfloat16*)gu, table, ids,
                                                                            sampled, num_sampled, req_of_token, top, experts, F,
-                                                                           vocab, weight, weights, code, p0, p1, err);
+                                                                           F_dense, vocab, weight, weights, dense_weight, code,
+                                                                           p0, p1, err);
     return xb_launch_status();
 }
 
@@ -288,13 +302,16 @@ XB_EXPORT int xb_expert_gather(int dtype, void* out, const void* x, const int* p
 }
 
 // ------------------------------------------------------------------------------------------
-// 3. combine.  out[t, :] = base[t, :] + sum_k w(t, k) * y[inv[t * top + k], :]   (a pair without a row adds nothing)
-// w(t, k) = weights[t * top + k], or 1 / top for all where no weights are given; base may be absent.
+// 3. combine.  out[t, :] = g(t) base[t, :] + sum_k w(t, k) * y[inv[t * top + k], :]   (a pair without a row adds nothing)
+// w(t, k) = weights[t * top + k], or 1 / top for all where no weights are given; base may be absent; g(t) = base_gate[t],
+// or 1 where no gate is given.
 // ------------------------------------------------------------------------------------------
 template <typename TO>
 __global__ void expert_combine_kernel(TO* __restrict__ out, const float* __restrict__ y, const int* __restrict__ inv, int top,
-                                      int N, float weight, const float* __restrict__ weights, const TO* __restrict__ base) {
+                                      int N, float weight, const float* __restrict__ weights, const TO* __restrict__ base,
+                                      const float* __restrict__ base_gate) {
     const int t = blockIdx.x;
+    const float bg = base_gate != nullptr ? base_gate[t] : 1.f;
     for (int c = threadIdx.x; c < N; c += blockDim.x) {
         float s = 0.f;
         for (int k = 0; k < top; ++k) {
@@ -302,7 +319,7 @@ __global__ void expert_combine_kernel(TO* __restrict__ out, const float* __restr
             if (r >= 0) s += (weights != nullptr ? weights[t * top + k] : 1.f) * y[(size_t)r * N + c];
         }
         s *= weight;
-        if (base != nullptr) s += to_f32<TO>(base[(size_t)t * N + c]);
+        if (base != nullptr) s = fmaf(bg, to_f32<TO>(base[(size_t)t * N + c]), s);
         out[(size_t)t * N + c] = from_f32<TO>(s);
     }
 }
@@ -311,8 +328,9 @@ __global__ void expert_combine_kernel(TO* __restrict__ out, const float* __restr
 // in the same order
 __global__ void expert_combine4_kernel(float4* __restrict__ out, const float4* __restrict__ y, const int* __restrict__ inv,
                                        int top, int N4, float weight, const float* __restrict__ weights,
-                                       const float4* __restrict__ base) {
+                                       const float4* __restrict__ base, const float* __restrict__ base_gate) {
     const int t = blockIdx.x;
+    const float bg = base_gate != nullptr ? base_gate[t] : 1.f;
     for (int c = threadIdx.x; c < N4; c += blockDim.x) {
         float4 s = make_float4(0.f, 0.f, 0.f, 0.f);
         for (int k = 0; k < top; ++k) {
@@ -325,23 +343,24 @@ __global__ void expert_combine4_kernel(float4* __restrict__ out, const float4* _
         s.x *= weight; s.y *= weight; s.z *= weight; s.w *= weight;
         if (base != nullptr) {
             const float4 bv = base[(size_t)t * N4 + c];
-            s.x += bv.x; s.y += bv.y; s.z += bv.z; s.w += bv.w;
+            s.x = fmaf(bg, bv.x, s.x); s.y = fmaf(bg, bv.y, s.y); s.z = fmaf(bg, bv.z, s.z); s.w = fmaf(bg, bv.w, s.w);
         }
         out[(size_t)t * N4 + c] = s;
     }
 }
 
 XB_EXPORT int xb_expert_combine(int out_dtype, void* out, const float* y, const int* inv, int tokens, int top, int N,
-                                const float* weights, const void* base, cudaStream_t stream) {
+                                const float* weights, const void* base, const float* base_gate, cudaStream_t stream) {
     if (tokens <= 0) return 0;
     const float weight = weights != nullptr ? 1.f : 1.f / (float)top;
     if (out_dtype == XB_F32 && N % 4 == 0 && !(((uintptr_t)out | (uintptr_t)y | (uintptr_t)base) & 15))
         expert_combine4_kernel<<<tokens, 256, 0, stream>>>((float4*)out, (const float4*)y, inv, top, N / 4, weight, weights,
-                                                           (const float4*)base);
+                                                           (const float4*)base, base_gate);
     else if (out_dtype == XB_F32)
-        expert_combine_kernel<float><<<tokens, 256, 0, stream>>>((float*)out, y, inv, top, N, weight, weights, (const float*)base);
+        expert_combine_kernel<float><<<tokens, 256, 0, stream>>>((float*)out, y, inv, top, N, weight, weights, (const float*)base,
+                                                         base_gate);
     else
         expert_combine_kernel<__nv_bfloat16><<<tokens, 256, 0, stream>>>((__nv_bfloat16*)out, y, inv, top, N, weight, weights,
-                                                                         (const __nv_bfloat16*)base);
+                                                                         (const __nv_bfloat16*)base, base_gate);
     return xb_launch_status();
 }

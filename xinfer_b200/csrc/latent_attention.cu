@@ -7,7 +7,8 @@
 // channels whose first kv_rank channels are also the value.  Here are the kernels around that attention:
 //
 //   latent_prepare_kernel   norms c, rotates k_r and writes the row [c | k_r] to its page; puts the query of
-//                           every head together as [q carried into the latent space | rotated q part]
+//                           every head together as [q carried into the latent space | rotated q part]; norms the
+//                           latent that the queries come from, where they have one
 //   gate_sigmoid_kernel     heads' outputs times sigmoid(gate), laid out token by token
 //   gemm_batched_plain      the per-head maps as a batch of small matrix products on FMA units (float32 path)
 #include "common.cuh"
@@ -16,7 +17,10 @@
 // [d plain | rd to rotate]) and, at kv_off, [kv_rank latent | rd key part] (kv_off < 0: this layer reads the
 // rows another layer wrote).  q_lat[t, h] (strides given) is the head's query already carried into the latent
 // space; absent: the latent part of q_abs has been written already (by the product that formed it) and stays.  The first `rot` channels of a rotated part turn by position * inv_freq[pair] (pairs 2i, 2i+1), cos
-// and sin times rot_mag; the others pass.
+// and sin times rot_mag; the others pass.  `tail` further channels of a query row, behind the rotated part, are zero
+// (cached rows that carry a key part this layer does not read).  nh = 0: no queries are put together.  A second row of
+// blocks (blockIdx.y = 1) norms the queries' own latent instead: cq[t] = the n_cq columns at cq_off, RMS-normed with
+// cq_w.
 template <typename T>
 __global__ void latent_prepare_kernel(T* __restrict__ q_abs, T* __restrict__ cache, const T* __restrict__ proj,
                                       long long row_len, int q_off, int kv_off, const T* __restrict__ q_lat,
@@ -24,9 +28,22 @@ __global__ void latent_prepare_kernel(T* __restrict__ q_abs, T* __restrict__ cac
                                       const float* __restrict__ inv_freq, const int* __restrict__ positions,
                                       const int* __restrict__ req_of_token, const int* __restrict__ block_table,
                                       int table_stride, int nh, int d, int rd, int rank, int rot, int page_size,
-                                      int num_pages, float eps, float rot_mag, int pairs, int* err) {
+                                      int num_pages, float eps, float rot_mag, int pairs, int tail, T* __restrict__ cq,
+                                      int cq_off, int n_cq, const float* __restrict__ cq_w, int* err) {
     extern __shared__ float sm[];
     __shared__ float scratch[33];
+    if (blockIdx.y == 1) {
+        const T* src = proj + (size_t)blockIdx.x * row_len + cq_off;
+        T* dst = cq + (size_t)blockIdx.x * n_cq;
+        float ss = 0.f;
+        for (int i = threadIdx.x; i < n_cq; i += blockDim.x) {
+            const float v = to_f32<T>(src[i]);
+            ss += v * v;
+        }
+        const float inv = 1.f / sqrtf(block_sum(ss, scratch) / (float)n_cq + eps);
+        for (int i = threadIdx.x; i < n_cq; i += blockDim.x) dst[i] = from_f32<T>(to_f32<T>(src[i]) * inv * cq_w[i]);
+        return;
+    }
     const int half = rot / 2;
     float* cs = sm;          // [half]
     float* sn = sm + half;   // [half]
@@ -41,8 +58,10 @@ __global__ void latent_prepare_kernel(T* __restrict__ q_abs, T* __restrict__ cac
     }
     __syncthreads();
     const T* row = proj + (size_t)t * row_len;
-    const int dk = rank + rd;
-    // queries: [latent part | rotated part]
+    const int dk = rank + rd + tail;
+    // queries: [latent part | rotated part | zeros]
+    for (int i = threadIdx.x; i < nh * tail; i += blockDim.x)
+        q_abs[((size_t)t * nh + i / tail) * dk + rank + rd + i % tail] = from_f32<T>(0.f);
     if (q_lat != nullptr) {
         for (int i = threadIdx.x; i < nh * rank; i += blockDim.x) {
             const int h = i / rank, c = i % rank;
@@ -106,10 +125,11 @@ XB_EXPORT int xb_latent_prepare(int dtype, void* q_abs, void* cache, const void*
                                 int kv_off, const void* q_lat, long long ql_ts, long long ql_hs, const float* norm_w,
                                 const float* inv_freq, const int* positions, const int* req_of_token,
                                 const int* block_table, int table_stride, int tokens, int nh, int d, int rd, int rank,
-                                int rot, int page_size, int num_pages, float eps, float rot_mag, int* err,
-                                cudaStream_t stream) {
+                                int rot, int page_size, int num_pages, float eps, float rot_mag, int tail, void* cq,
+                                int cq_off, int n_cq, const float* cq_w, int* err, cudaStream_t stream) {
     if (tokens <= 0) return 0;
-    if (rot % 2 || rot > rd) return (int)cudaErrorInvalidValue;
+    // a layer that writes rows writes whole ones
+    if (rot % 2 || rot > rd || (tail > 0 && kv_off >= 0)) return (int)cudaErrorInvalidValue;
     const size_t smem = (size_t)rot * sizeof(float);
     if (smem > 48 * 1024) return (int)cudaErrorInvalidValue;
     const int work = q_lat != nullptr ? nh * (rank + rd) : (nh * rd > rank + rd ? nh * rd : rank + rd);
@@ -117,10 +137,10 @@ XB_EXPORT int xb_latent_prepare(int dtype, void* q_abs, void* cache, const void*
     // sum), so many resident blocks hide more than many threads per block
     const int threads = work >= 16384 ? 256 : 128;
 #define XB_GO(T)                                                                                                        \
-    latent_prepare_kernel<T><<<tokens, threads, smem, stream>>>((T*)q_abs, (T*)cache, (const T*)proj, row_len, q_off,  \
+    latent_prepare_kernel<T><<<dim3(tokens, cq != nullptr ? 2 : 1), threads, smem, stream>>>((T*)q_abs, (T*)cache, (const T*)proj, row_len, q_off,  \
         kv_off, (const T*)q_lat, ql_ts, ql_hs, norm_w, inv_freq, positions, req_of_token, block_table, table_stride,   \
-        nh, d, rd, rank, rot, page_size, num_pages, eps, rot_mag, pairs, err)
-    const int pairs = (dtype == XB_BF16 && !((row_len | q_off | d | rd | rank) & 1) &&
+        nh, d, rd, rank, rot, page_size, num_pages, eps, rot_mag, pairs, tail, (T*)cq, cq_off, n_cq, cq_w, err)
+    const int pairs = (dtype == XB_BF16 && !((row_len | q_off | d | rd | rank | tail) & 1) &&
                        !(((uintptr_t)proj | (uintptr_t)q_abs) & 3)) ? 1 : 0;
     if (dtype == XB_F32) XB_GO(float);
     else XB_GO(__nv_bfloat16);

@@ -3,9 +3,11 @@
 //   selective_scan_kernel   (state-space duality)   S[N, P]:  S <- exp(-A dt) S + dt B x^T,   y = S^T C + D x
 //   delta_rule_kernel       (gated delta rule)      S[d, dv]: S <- diag(g) S,  u = beta (v - S^T k),  S <- S + k u^T,
 //                                                             o = S^T q      (read after the token's own update)    
+//   linear_scan_kernel      (gated linear attention)  S[d, dv]: S <- diag(alpha) S + k v^T,  o = scale S^T q
+//   low_rank_decay_kernel   alpha = sigmoid(W_a2 low + b)^(1 / tau) for it, per token and key channel
 //   gated_head_norm_kernel  the gate and the RMS norm over a head (or a group of channels) behind either
 //
-// Layout of both scans: a block takes one (request, head) and a tile of the state's columns (columns never mix).
+// Layout of the scans: a block takes one (request, head) and a tile of the state's columns (columns never mix).
 // Its first warps compute: a lane keeps kRows rows of two neighbouring columns in registers; DS lanes of a warp
 // share a column pair and fold their sums over rows with shuffles.  Its last warps feed them: tokens of a request
 // are walked in order, a tile of TT tokens at a time, and while the computing warps work on one tile the feeding
@@ -366,6 +368,149 @@ __global__ void __launch_bounds__(384, 1) delta_rule_kernel(float* __restrict__ 
     }
 }
 
+// proj[t] holds q (H*d from column 0), k (H*d behind it) and v (H*dv behind that) of a token; alpha[t] the decay of
+// every (head, key channel).  state [slots, H, d, dv].  o [T, H*dv] = scale * S^T q after the token's own write.  Shared
+// memory: two stages of q[TT][DP] k[TT][DP] alpha[TT][DP] v[TT][VT], then two tiles o[TT][VT].
+template <int DS>
+__global__ void __launch_bounds__(384, 1) linear_scan_kernel(float* __restrict__ o, const float* __restrict__ proj,
+                                                             long long ldp, const float* __restrict__ alpha,
+                                                             float* __restrict__ state, const int* __restrict__ q_start,
+                                                             const int* __restrict__ slots, int H, int d, int dv, float scale,
+                                                             int TT, int stage, int cw, int vec) {
+    extern __shared__ __align__(16) float scan_smem[];
+    constexpr int CGW = 32 / DS, DP = DS * kRowsPad, NR = DS * kRows;
+    const int b = blockIdx.x, h = blockIdx.y;
+    const int lane = threadIdx.x & 31, w = threadIdx.x >> 5;
+    const int VT = cw * CGW * 2, c_base = blockIdx.z * VT;
+    const int slot = slots[b];
+    const int t0 = q_start[b], t1 = q_start[b + 1];
+    if (slot < 0 || t1 <= t0) return;
+    const int ntiles = (t1 - t0 + TT - 1) / TT;
+    float* so = scan_smem + 2 * stage;
+    if (w >= cw) {
+        // feeding warps: warp `pi` of `pw` takes tokens pi, pi + pw, ... of every tile
+        const int pi = w - cw, pw = (blockDim.x >> 5) - cw;
+        auto bring = [&](int tile) {
+            float* sq = scan_smem + (tile & 1) * stage;
+            float* sk = sq + TT * DP;
+            float* sa = sk + TT * DP;
+            float* sv = sa + TT * DP;
+            const int tb = t0 + tile * TT, nt = min(TT, t1 - tb);
+            for (int tt = pi; tt < nt; tt += pw) {
+                const float* row = proj + (size_t)(tb + tt) * ldp;
+                stage_rows(sq + tt * DP, row + h * d, d, NR, lane, vec);
+                stage_rows(sk + tt * DP, row + (H + h) * d, d, NR, lane, vec);
+                stage_rows(sa + tt * DP, alpha + ((size_t)(tb + tt) * H + h) * d, d, NR, lane, vec);
+                stage_cols(sv + tt * VT, row + 2 * H * d + h * dv, c_base, dv, VT, lane, vec);
+            }
+            scan_cp_land();
+        };
+        auto leave = [&](int tile) {
+            const float* src = so + (tile & 1) * TT * VT;
+            const int tb = t0 + tile * TT, nt = min(TT, t1 - tb);
+            for (int tt = pi; tt < nt; tt += pw)
+                for (int c = lane; c < VT; c += 32)
+                    if (c_base + c < dv) o[((size_t)(tb + tt) * H + h) * dv + c_base + c] = src[tt * VT + c];
+        };
+        bring(0);
+        __syncthreads();
+        for (int tile = 0; tile < ntiles; ++tile) {
+            if (tile + 1 < ntiles) bring(tile + 1);
+            if (tile > 0) leave(tile - 1);
+            __syncthreads();
+        }
+        leave(ntiles - 1);
+        return;
+    }
+    const int ds = lane / CGW, cl = (w * CGW + lane % CGW) * 2, v0 = c_base + cl;
+    float S0[kRows], S1[kRows];
+    float* st = state + ((size_t)slot * H + h) * d * dv;
+#pragma unroll
+    for (int r = 0; r < kRows; ++r) {
+        const int j = ds * kRows + r;
+        S0[r] = (j < d && v0 < dv) ? st[(size_t)j * dv + v0] : 0.f;
+        S1[r] = (j < d && v0 + 1 < dv) ? st[(size_t)j * dv + v0 + 1] : 0.f;
+    }
+    __syncthreads();
+    for (int tile = 0; tile < ntiles; ++tile) {
+        const float* sq = scan_smem + (tile & 1) * stage + ds * kRowsPad;
+        const float* sk = sq + TT * DP;
+        const float* sa = sk + TT * DP;
+        const float* sv = scan_smem + (tile & 1) * stage + 3 * TT * DP + cl;
+        float* out = so + (tile & 1) * TT * VT + cl;
+        const int nt = min(TT, t1 - t0 - tile * TT);
+        for (int tt = 0; tt < nt; ++tt, sq += DP, sk += DP, sa += DP, sv += VT, out += VT) {
+            const float2 vv = *reinterpret_cast<const float2*>(sv);
+            const float4* qp = reinterpret_cast<const float4*>(sq);
+            const float4* kp = reinterpret_cast<const float4*>(sk);
+            const float4* ap = reinterpret_cast<const float4*>(sa);
+            float a0 = 0.f, a1 = 0.f;
+#pragma unroll
+            for (int i = 0; i < kRows / 4; ++i) {
+                const float4 q4 = qp[i], k4 = kp[i], g4 = ap[i];
+                const float qq[4] = {q4.x, q4.y, q4.z, q4.w}, kq[4] = {k4.x, k4.y, k4.z, k4.w};
+                const float gq[4] = {g4.x, g4.y, g4.z, g4.w};
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                    const int r = 4 * i + e;
+                    S0[r] = fmaf(gq[e], S0[r], kq[e] * vv.x);
+                    S1[r] = fmaf(gq[e], S1[r], kq[e] * vv.y);
+                    a0 = fmaf(S0[r], qq[e], a0);
+                    a1 = fmaf(S1[r], qq[e], a1);
+                }
+            }
+            a0 = fold_rows<DS>(a0);
+            a1 = fold_rows<DS>(a1);
+            if (ds == 0) *reinterpret_cast<float2*>(out) = make_float2(scale * a0, scale * a1);
+        }
+        __syncthreads();
+    }
+#pragma unroll
+    for (int r = 0; r < kRows; ++r) {
+        const int j = ds * kRows + r;
+        if (j < d && v0 < dv) st[(size_t)j * dv + v0] = S0[r];
+        if (j < d && v0 + 1 < dv) st[(size_t)j * dv + v0 + 1] = S1[r];
+    }
+}
+
+// alpha[t, c] = sigmoid(z)^(1 / tau) = exp(-softplus(-z) / tau),  z = bias[c] + sum_r w[c, r] low[t, r].  low is a
+// column range of wider float32 rows.  A thread per channel and a tile of tokens; r in order for every output.
+constexpr int kDecayTokens = 8, kDecayRanks = 32;
+__global__ void __launch_bounds__(128) low_rank_decay_kernel(float* __restrict__ alpha, const float* __restrict__ low,
+                                                             long long ldl, const float* __restrict__ w,
+                                                             const float* __restrict__ bias, int tokens, int C, int R,
+                                                             float inv_tau) {
+    __shared__ float sl[kDecayRanks][kDecayTokens];
+    const int tb = blockIdx.x * kDecayTokens, nt = min(kDecayTokens, tokens - tb);
+    const int c = blockIdx.y * blockDim.x + threadIdx.x;
+    float z[kDecayTokens];
+    const float b = c < C ? bias[c] : 0.f;
+#pragma unroll
+    for (int i = 0; i < kDecayTokens; ++i) z[i] = b;
+    for (int r0 = 0; r0 < R; r0 += kDecayRanks) {
+        const int nr = min(kDecayRanks, R - r0);
+        if (r0 > 0) __syncthreads();
+        for (int i = threadIdx.x; i < kDecayRanks * kDecayTokens; i += blockDim.x) {
+            const int tt = i / kDecayRanks, r = i % kDecayRanks;
+            sl[r][tt] = (tt < nt && r < nr) ? low[(size_t)(tb + tt) * ldl + r0 + r] : 0.f;
+        }
+        __syncthreads();
+        if (c < C) {
+            const float* wr = w + (size_t)c * R + r0;
+#pragma unroll 8
+            for (int r = 0; r < nr; ++r) {
+                const float wv = wr[r];
+#pragma unroll
+                for (int i = 0; i < kDecayTokens; ++i) z[i] = fmaf(wv, sl[r][i], z[i]);
+            }
+        }
+    }
+    if (c >= C) return;
+#pragma unroll
+    for (int i = 0; i < kDecayTokens; ++i)
+        if (i < nt) alpha[(size_t)(tb + i) * C + c] = expf(-softplus_f32(-z[i]) * inv_tau);
+}
+
 // Row groups per column pair: the smallest power of two with DS * kRows >= rows.
 static inline int scan_row_groups(int rows) {
     int ds = 1;
@@ -458,9 +603,36 @@ XB_EXPORT int xb_delta_rule(float* o, const float* qkv, int Cq, const float* pro
     return xb_launch_status();
 }
 
+XB_EXPORT int xb_linear_scan(float* o, const float* proj, long long ldp, const float* alpha, float* state, const int* q_start,
+                             const int* slots, int entries, int H, int d, int dv, float scale, cudaStream_t stream) {
+    if (entries <= 0) return 0;
+    if (d < 1 || d > 32 * kRows || dv < 1 || H < 1 || H > 65535) return (int)cudaErrorInvalidValue;
+    const int ds = scan_row_groups(d);
+    const int warps = scan_warps(dv, ds, (long long)entries * H);
+    const int vt = warps * (32 / ds) * 2;
+    int tt, stage;
+    size_t bytes;
+    scan_tile(3, ds, vt, tt, stage, bytes);
+    const dim3 grid(entries, H, (dv + vt - 1) / vt);
+    const int threads = (warps + 4) * 32;  // four feeding warps: they only copy
+    const int vec = scan_aligned16(proj) && scan_aligned16(alpha) && ldp % 4 == 0 && d % 4 == 0 && dv % 4 == 0 && vt % 4 == 0;
+    XB_SCAN_DISPATCH(linear_scan_kernel, ds, o, proj, ldp, alpha, state, q_start, slots, H, d, dv, scale, tt, stage, warps, vec)
+    return xb_launch_status();
+}
+
+XB_EXPORT int xb_low_rank_decay(float* alpha, const float* low, long long ldl, const float* w, const float* bias, int tokens,
+                                int C, int R, float tau, cudaStream_t stream) {
+    if (tokens <= 0 || C <= 0) return 0;
+    if (R < 1 || !(tau > 0.f) || (C + 127) / 128 > 65535) return (int)cudaErrorInvalidValue;
+    const dim3 grid((tokens + kDecayTokens - 1) / kDecayTokens, (C + 127) / 128);
+    low_rank_decay_kernel<<<grid, 128, 0, stream>>>(alpha, low, ldl, w, bias, tokens, C, R, 1.f / tau);
+    return xb_launch_status();
+}
+
 // One block per (token, group of `part` consecutive channels of the W):
 //   mode 0:  v = y * silu(gate);  out = v * rsqrt(mean(v^2) + eps) * w[c mod w_len]          (gate before the norm)
 //   mode 1:  out = y * rsqrt(mean(y^2) + eps) * w[c mod w_len] * sigmoid(gate)               (gate behind it)
+//   mode 2:  the same with silu(gate)
 // gate is column g_off + c of a wider float32 row.
 template <typename TO>
 __global__ void gated_head_norm_kernel(TO* __restrict__ out, const float* __restrict__ y, const float* __restrict__ gate,
@@ -487,7 +659,7 @@ __global__ void gated_head_norm_kernel(TO* __restrict__ out, const float* __rest
         if (mode == 0)
             v = v * (z / (1.f + expf(-z))) * inv * w[(c0 + i) % w_len];
         else
-            v = v * inv * w[(c0 + i) % w_len] * sigmoid_exact(z);
+            v = v * inv * w[(c0 + i) % w_len] * (mode == 2 ? z * sigmoid_exact(z) : sigmoid_exact(z));
         o[i] = from_f32<TO>(v);
     }
 }
@@ -524,7 +696,7 @@ __global__ void __launch_bounds__(256) gated_head_norm_warp_kernel(TO* __restric
         const int i = lane + 32 * k;
         if (i >= part) continue;
         float r = v[k] * inv * w[(c0 + i) % w_len];
-        if (mode != 0) r *= sigmoid_exact(z[k]);
+        if (mode != 0) r *= mode == 2 ? z[k] * sigmoid_exact(z[k]) : sigmoid_exact(z[k]);
         o[i] = from_f32<TO>(r);
     }
 }

@@ -868,13 +868,16 @@ def expert_gemm(y, a, w, offsets, perm, gather: bool, top: int, gated: bool, *, 
                 activation: str = "silu", params=()):
     """y[r] = a[src(r)] . w[e(r)]^T over rows grouped by expert (``expert_route``).  ``w`` is
     ``[experts, N, K]`` (``[experts, 2 N, K]`` when ``gated``: y = act(gate) * f(up), ``activation``), or with
-    ``side_by_side`` ``[N, experts * K]``: the experts' matrices beside each other along K."""
+    ``side_by_side`` ``[N, experts * K + more]``: the experts' matrices beside each other along K (K is then ``a``'s),
+    other columns behind them."""
     rows = y.shape[0]
     if side_by_side:
         E = offsets.numel() - 1
-        N, K = w.shape[0], w.shape[1] // E
-        _need(w, "w", a.dtype, (N, E * K))
-        ldw, estride = E * K, K
+        N, K = w.shape[0], a.shape[1]
+        _need(w, "w", a.dtype, (N, None))
+        if w.shape[1] < E * K:
+            raise KernelError(f"{E} matrices of {K} columns do not fit beside each other in {w.shape[1]}")
+        ldw, estride = w.shape[1], K
     else:
         E = w.shape[0]
         N = w.shape[1] // (2 if gated else 1)
@@ -897,24 +900,30 @@ def expert_gemm(y, a, w, offsets, perm, gather: bool, top: int, gated: bool, *, 
 
 
 def expert_select_gate(act, gu, table, ids, sampled, req_of_token, top: int, experts: int, err, *, weights=None,
-                       activation: str = "silu", params=()):
+                       activation: str = "silu", params=(), dense: int = 0, dense_weight=None):
     """From every expert's gate/up values of every token, ``gu [T, experts * 2 F]``, the inputs of the down
     product with the experts side by side: ``act [T, experts * F]`` holds ``silu(gate) * up / top`` for a
     token's own experts and zero for the others.  ``ids`` None: ``table`` has a row per token of the step;
     ``weights`` (float32, like ``table``): a chosen expert's own weight instead of 1 / top; ``activation`` as in
-    ``swiglu``."""
+    ``swiglu``.  ``dense`` > 0: behind the experts every row holds the gate and up halves of one more feed-forward of
+    that width, which every token runs with its ``dense_weight`` (float32 ``[T]``)."""
     T = gu.shape[0]
+    if dense:
+        _need(dense_weight, "dense_weight", torch.float32)
+        if dense_weight.numel() < T:
+            raise KernelError(f"dense_weight holds {dense_weight.numel()} numbers for {T} tokens")
     code, p0, p1 = activation_args(activation, params)
     if weights is not None:
         _need(weights, "weights", torch.float32, tuple(table.shape))
-    Fdim = gu.shape[1] // (2 * experts)
-    _need(gu, "gu", None, (T, experts * 2 * Fdim))
-    _need(act, "act", gu.dtype, (T, experts * Fdim))
+    Fdim = (gu.shape[1] - 2 * dense) // (2 * experts)
+    _need(gu, "gu", None, (T, 2 * (experts * Fdim + dense)))
+    _need(act, "act", gu.dtype, (T, experts * Fdim + dense))
     _need(table, "table", torch.int32, (None, top))
     _ok(kernels_lib().xb_expert_select_gate(dtype_code(gu.dtype), act.data_ptr(), gu.data_ptr(), table.data_ptr(), _ptr(ids),
                                             _ptr(sampled), sampled.numel() if sampled is not None else 0,
-                                            req_of_token.data_ptr(), T, int(top), int(experts), Fdim, table.shape[0],
-                                            _ptr(weights), code, p0, p1, err.data_ptr(), _stream()), "expert_select_gate")
+                                            req_of_token.data_ptr(), T, int(top), int(experts), Fdim, int(dense), table.shape[0],
+                                            _ptr(weights), _ptr(dense_weight), code, p0, p1, err.data_ptr(), _stream()),
+        "expert_select_gate")
 
 
 def expert_gather(out, x, perm, offsets, top: int):
@@ -926,9 +935,10 @@ def expert_gather(out, x, perm, offsets, top: int):
                                        rows, int(top), offsets.numel() - 1, K, _stream()), "expert_gather")
 
 
-def expert_combine(out, y, inv, top: int, *, weights=None, base=None):
+def expert_combine(out, y, inv, top: int, *, weights=None, base=None, base_gate=None):
     """out[t] = base[t] + sum_k w(t, k) y[inv[t, k]]: a token's experts summed in the order of k, each times its own
-    weight (``weights`` float32 ``[T, top]``) or all times 1 / top; ``base`` (like ``out``, may be ``out``) is added."""
+    weight (``weights`` float32 ``[T, top]``) or all times 1 / top; ``base`` (like ``out``, may be ``out``) is added,
+    times ``base_gate`` (float32 ``[T]``) where that is given."""
     T, N = out.shape
     _need(y, "y", torch.float32, (None, N))
     _need(out, "out", None, (T, N))
@@ -936,57 +946,80 @@ def expert_combine(out, y, inv, top: int, *, weights=None, base=None):
         _need(weights, "weights", torch.float32, (T, top))
     if base is not None:
         _need(base, "base", out.dtype, (T, N))
+    if base_gate is not None:
+        _need(base_gate, "base_gate", torch.float32, (T,))
     _ok(kernels_lib().xb_expert_combine(dtype_code(out.dtype), out.data_ptr(), y.data_ptr(), inv.data_ptr(), T, int(top), N,
-                                        _ptr(weights), _ptr(base), _stream()), "expert_combine")
+                                        _ptr(weights), _ptr(base), _ptr(base_gate), _stream()), "expert_combine")
 
 
 def expert_router(choice, weight, h, w_router, correction, req_of_token, top: int, groups: int = 1, keep: int = 1,
-                  group_best: int = 2, renormalize: bool = False):
-    """A sigmoid router: scores ``s = sigmoid(W_r h)`` in float32, choice scores ``s + correction``; only experts of
+                  group_best: int = 2, renormalize: bool = False, *, softmax: bool = False, renormalize_eps: float = 0.0,
+                  weight_scale: float = 1.0, gate=None):
+    """A router: scores ``s = sigmoid(W_r h)`` (``softmax``: over all experts) in float32, choice scores
+    ``s + correction``; only experts of
     the ``keep`` best of ``groups`` equal groups of neighbours can be chosen (a group's score: the sum of its
     ``group_best`` largest choice scores); ``choice [T, top]`` (int32) receives the experts with the largest choice
-    scores and ``weight [T, top]`` their plain scores (divided by their sum with ``renormalize``)."""
+    scores and ``weight [T, top]`` their plain scores (with ``renormalize`` divided by their sum plus
+    ``renormalize_eps``) times ``weight_scale``.  ``gate`` (float32 ``[T]``): receives the sigmoid of the product with
+    one more row of ``w_router`` behind the experts'."""
     T, K = h.shape
-    E = w_router.shape[0]
+    E = w_router.shape[0] - (gate is not None)
     _need(h, "h", None, (T, K))
-    _need(w_router, "w_router", torch.float32, (E, K))
+    _need(w_router, "w_router", torch.float32, (None, K))
+    if gate is not None:
+        _need(gate, "gate", torch.float32, (T,))
     _need(choice, "choice", torch.int32, (T, top))
     _need(weight, "weight", torch.float32, (T, top))
     if correction is not None:
         _need(correction, "correction", torch.float32, (E,))
     _ok(kernels_lib().xb_expert_router(dtype_code(h.dtype), choice.data_ptr(), weight.data_ptr(), h.data_ptr(),
-                                       w_router.data_ptr(), _ptr(correction), req_of_token.data_ptr(), T, E, K, int(top),
-                                       int(groups), int(keep), int(group_best), int(bool(renormalize)), _stream()),
+                                       w_router.data_ptr(), _ptr(correction), req_of_token.data_ptr(), _ptr(gate), T, E, K,
+                                       int(top), int(groups), int(keep), int(group_best), int(bool(softmax)),
+                                       int(bool(renormalize)), float(renormalize_eps), float(weight_scale), _stream()),
         "expert_router")
 
 
 # ---- attention over a cached latent ---------------------------------------------------------------------------------
 def latent_prepare(q_abs, cache, proj, q_off, kv_off, q_lat, norm_w, inv_freq, positions, req_of_token, block_table,
-                   table_stride, nh, d, rd, rank, rot, eps, rot_magnitude, err):
+                   table_stride, nh, d, rd, rank, rot, eps, rot_magnitude, err, *, tail: int = 0, query_latent=None):
     """Per token of the packed projection ``proj``: the query of every head as ``q_abs[t, h] = [q_lat[h, t] | rotated
     rd channels]`` (``q_lat`` ``[heads, T, rank]``: the plain query part carried into the latent space; None: the
-    product that formed it has written it into ``q_abs`` already), and, with
+    product that formed it has written it into ``q_abs`` already; ``nh`` 0: no queries), and, with
     ``kv_off`` >= 0, the cached row ``[RMS-normed rank channels * norm_w | rotated rd channels]`` into its page
     (``cache`` ``[page, slot, rank + rd]``).  Rotation: pairs (2i, 2i + 1) of the first ``rot`` channels by
-    ``position * inv_freq[i]``, cos and sin times ``rot_magnitude``."""
+    ``position * inv_freq[i]``, cos and sin times ``rot_magnitude``.  ``tail``: further channels of the cached rows that
+    this layer does not read; a query row ends in as many zeros.  ``query_latent`` = (out ``[T, n]``, column, weight):
+    out receives the n columns of ``proj`` from that column on, RMS-normed times the weight."""
     T = proj.shape[0]
+    width = rank + rd + tail
     _need(proj, "proj", None, (T, None))
-    _need(q_abs, "q_abs", proj.dtype, (T, nh, rank + rd))
+    if nh:
+        _need(q_abs, "q_abs", proj.dtype, (T, nh, width))
+        if q_off + nh * (d + rd) > proj.shape[1]:
+            raise KernelError("the queries lie outside the projection's rows")
     if q_lat is not None:
         _need(q_lat, "q_lat", proj.dtype, (nh, T, rank))
-    _need(cache, "cache", proj.dtype, (None, None, rank + rd))
-    _need(inv_freq, "inv_freq", torch.float32, (rot // 2,))
+    _need(cache, "cache", proj.dtype, (None, None, width))
+    if rot:
+        _need(inv_freq, "inv_freq", torch.float32, (rot // 2,))
     if kv_off >= 0:
         _need(norm_w, "norm_w", torch.float32, (rank,))
         if kv_off + rank + rd > proj.shape[1]:
             raise KernelError("the latent part lies outside the projection's rows")
-    if q_off + nh * (d + rd) > proj.shape[1]:
-        raise KernelError("the queries lie outside the projection's rows")
+        if tail:
+            raise KernelError("a layer that writes rows reads all their channels")
+    cq, cq_off, cq_w = query_latent if query_latent is not None else (None, 0, None)
+    if cq is not None:
+        _need(cq, "query latent", proj.dtype, (T, None))
+        _need(cq_w, "query latent's weight", torch.float32, (cq.shape[1],))
+        if cq_off < 0 or cq_off + cq.shape[1] > proj.shape[1]:
+            raise KernelError("the queries' latent lies outside the projection's rows")
     _ok(kernels_lib().xb_latent_prepare(
-        dtype_code(proj.dtype), q_abs.data_ptr(), cache.data_ptr(), proj.data_ptr(), proj.shape[1], int(q_off), int(kv_off),
-        _ptr(q_lat), rank, T * rank, _ptr(norm_w), inv_freq.data_ptr(), positions.data_ptr(), req_of_token.data_ptr(),
+        dtype_code(proj.dtype), _ptr(q_abs), cache.data_ptr(), proj.data_ptr(), proj.shape[1], int(q_off), int(kv_off),
+        _ptr(q_lat), rank, T * rank, _ptr(norm_w), _ptr(inv_freq), positions.data_ptr(), req_of_token.data_ptr(),
         block_table.data_ptr(), int(table_stride), T, nh, d, rd, rank, int(rot), cache.shape[1], cache.shape[0], float(eps),
-        float(rot_magnitude), err.data_ptr(), _stream()), "latent_prepare")
+        float(rot_magnitude), int(tail), _ptr(cq), int(cq_off), cq.shape[1] if cq is not None else 0, _ptr(cq_w),
+        err.data_ptr(), _stream()), "latent_prepare")
 
 
 def attn_latent_mma_takes(dk: int, rank: int) -> bool:
@@ -1234,9 +1267,84 @@ def delta_rule(o, qkv, proj, beta_off, ag, dt_bias, a_log, state, q_start, slots
                                     float(unit_eps), _stream()), "delta_rule")
 
 
-def gated_head_norm(out, y, gate, g_off, weight, part, eps, gate_after: bool):
+def linear_scan(o, proj, alpha, state, q_start, slots, num_entries, heads, d, dv, scale: float):
+    """Gated linear attention per (request, head): S <- diag(alpha) S + k v^T, o = scale * S^T q after the token's own
+    write.  ``proj`` float32 rows ``[q | k | v | ...]``, ``alpha`` float32 ``[T, heads * d]``, ``state``
+    ``[slots, heads, d, dv]``; ``o`` ``[T, heads * dv]`` before its norm and gate."""
+    T = proj.shape[0]
+    _need(proj, "proj", torch.float32, (T, None))
+    if proj.shape[1] < heads * (2 * d + dv):
+        raise KernelError("q, k and v lie outside the projection's rows")
+    _need(alpha, "alpha", torch.float32, (T, heads * d))
+    _need(o, "o", torch.float32, (T, heads * dv))
+    _need(state, "state", torch.float32, (None, heads, d, dv))
+    _ok(kernels_lib().xb_linear_scan(o.data_ptr(), proj.data_ptr(), proj.shape[1], alpha.data_ptr(), state.data_ptr(),
+                                     q_start.data_ptr(), slots.data_ptr(), int(num_entries), heads, d, dv, float(scale),
+                                     _stream()), "linear_scan")
+
+
+def low_rank_decay(alpha, low, w, bias, tau: float):
+    """alpha[t, c] = sigmoid(bias[c] + w[c] . low[t])^(1 / tau), float32 throughout; ``low`` ``[T, rank]`` may be a column
+    range of wider float32 rows."""
+    T, C = alpha.shape
+    R = w.shape[1]
+    _need(alpha, "alpha", torch.float32, (T, C))
+    _need(w, "w", torch.float32, (C, R))
+    _need(bias, "bias", torch.float32, (C,))
+    if low.dtype != torch.float32 or tuple(low.shape) != (T, R) or low.stride(1) != 1 or not low.is_cuda:
+        raise KernelError("low must be a float32 CUDA view [T, rank] with unit column stride")
+    _ok(kernels_lib().xb_low_rank_decay(alpha.data_ptr(), low.data_ptr(), low.stride(0), w.data_ptr(), bias.data_ptr(), T, C, R,
+                                        float(tau), _stream()), "low_rank_decay")
+
+
+# taps up to which the sum of a branch is formed by the convolution's own kernel
+STREAM_CONV_FUSED_TAPS = 8
+
+
+def stream_conv(out, x, taps, state, req_of_token, q_start, slots, num_entries, *, branch=None, branch_weight=None,
+                branch_eps: float = 0.0, branch_offset: float = 0.0, branch_scale: float = 1.0, sum_out=None,
+                single: bool = False):
+    """out[t] = s[t] + sum_j taps[:, j] * s[t - (K-1) + j] per request, with s = x (+ branch_scale * branch, or times the
+    branch's RMS norm ``branch / rms(branch) * (branch_offset + branch_weight)``), all float32 but ``out`` (either type).
+    ``sum_out`` (not ``x``) receives s where there is a branch.  The K-1 sums before a step's first token come from
+    ``state`` ``[slots, K-1, C]``, which then receives the step's last K-1 sums - in the same launch where every request
+    brings one token (``single``)."""
+    T, C = x.shape
+    K = taps.shape[1]
+    _need(x, "x", torch.float32, (T, C))
+    _need(out, "out", None, (T, C))
+    _need(taps, "taps", torch.float32, (C, K))
+    if K > CONV_MAX_TAPS:
+        raise KernelError(f"a short convolution has at most {CONV_MAX_TAPS} taps, got {K}")
+    if K > 1:
+        _need(state, "state", torch.float32, (None, K - 1, C))
+    if branch is not None:
+        if K > STREAM_CONV_FUSED_TAPS:
+            raise KernelError(f"a branch is summed for up to {STREAM_CONV_FUSED_TAPS} taps, got {K}")
+        _need(branch, "branch", torch.float32, (T, C))
+        _need(sum_out, "sum_out", torch.float32, (T, C))
+        if branch_weight is not None:
+            _need(branch_weight, "branch_weight", torch.float32, (C,))
+        if sum_out.data_ptr() in (x.data_ptr(), branch.data_ptr()):
+            raise KernelError("the sum needs a buffer of its own")
+    elif branch_weight is not None or sum_out is not None:
+        raise KernelError("a branch norm or a stored sum needs a branch")
+    in_pass = bool(single) and K <= STREAM_CONV_FUSED_TAPS
+    lib = kernels_lib()
+    _ok(lib.xb_stream_conv(dtype_code(out.dtype), out.data_ptr(), _ptr(sum_out), x.data_ptr(), _ptr(branch), _ptr(branch_weight),
+                           taps.data_ptr(), _ptr(state) if K > 1 else None, req_of_token.data_ptr(), q_start.data_ptr(),
+                           slots.data_ptr(), T, C, K, float(branch_eps), float(branch_offset), float(branch_scale), int(in_pass),
+                           _stream()), "stream_conv")
+    if K > 1 and not in_pass:
+        s = x if sum_out is None else sum_out
+        _ok(lib.xb_conv_state(state.data_ptr(), s.data_ptr(), C, 0, q_start.data_ptr(), slots.data_ptr(), int(num_entries), C, K,
+                              _stream()), "conv_state")
+
+
+def gated_head_norm(out, y, gate, g_off, weight, part, eps, gate_after: bool, silu_gate: bool = False):
     """Per token and group of ``part`` channels of ``y`` (float32): with ``gate_after`` False,
-    v = y * silu(gate), out = v / rms(v) * weight; with True, out = y / rms(y) * weight * sigmoid(gate).  ``gate`` is
+    v = y * silu(gate), out = v / rms(v) * weight; with True, out = y / rms(y) * weight * sigmoid(gate), or silu(gate)
+    for the last factor with ``silu_gate``.  ``gate`` is
     the columns from ``g_off`` of float32 rows; ``weight`` repeats every ``weight.numel()`` channels."""
     T, W = y.shape
     _need(y, "y", torch.float32, (T, W))
@@ -1247,4 +1355,4 @@ def gated_head_norm(out, y, gate, g_off, weight, part, eps, gate_after: bool):
         raise KernelError("gate columns, group size or weight length do not fit the rows")
     _ok(kernels_lib().xb_gated_head_norm(dtype_code(out.dtype), out.data_ptr(), y.data_ptr(), gate.data_ptr(), gate.shape[1],
                                          int(g_off), weight.data_ptr(), weight.numel(), T, W, int(part), float(eps),
-                                         int(bool(gate_after)), _stream()), "gated_head_norm")
+                                         (2 if silu_gate else 1) if gate_after else 0, _stream()), "gated_head_norm")

@@ -129,9 +129,13 @@ def _declare_kernels(lib):
     _sig(lib, "xb_conv_state", I, [P, P, L, I, P, P, I, I, I, P])
     _sig(lib, "xb_selective_scan", I, [P, P, I, P, L, I, P, P, P, P, P, P, I, I, I, I, I, P])
     _sig(lib, "xb_delta_rule", I, [P, P, I, P, L, I, P, L, P, P, P, P, P, I, I, I, I, I, F, P])
+    _sig(lib, "xb_linear_scan", I, [P, P, L, P, P, P, P, I, I, I, I, F, P])
+    _sig(lib, "xb_low_rank_decay", I, [P, P, L, P, P, I, I, I, F, P])
+    _sig(lib, "xb_stream_conv", I, [I, P, P, P, P, P, P, P, P, P, P, I, I, I, F, F, F, I, P])
     _sig(lib, "xb_gated_head_norm", I, [I, P, P, P, L, I, P, I, I, I, I, F, I, P])
     _sig(lib, "xb_dyt_norm", I, [I, I, I, P, P, P, P, P, P, P, P, F, P, P, P, I, I, I, P, P])
-    _sig(lib, "xb_latent_prepare", I, [I, P, P, P, L, I, I, P, L, L, P, P, P, P, P, I, I, I, I, I, I, I, I, I, F, F, P, P])
+    _sig(lib, "xb_latent_prepare", I,
+         [I, P, P, P, L, I, I, P, L, L, P, P, P, P, P, I, I, I, I, I, I, I, I, I, F, F, I, P, I, I, P, P, P])
     _sig(lib, "xb_attn_latent_mma_takes", I, [I, I])
     _sig(lib, "xb_attn_latent_mma", I, [P, P, P, P, P, I, P, I, I, I, I, I, I, I, I, F, P, I, I, P, P, P, P])
     _sig(lib, "xb_gate_sigmoid", I, [I, P, P, L, L, P, L, I, I, I, I, P])
@@ -144,9 +148,9 @@ def _declare_kernels(lib):
     _sig(lib, "xb_polynorm", I, [I, P, P, P, I, I, F, P])
     _sig(lib, "xb_expert_route", I, [P, P, P, P, P, P, I, P, I, I, I, I, P, P])
     _sig(lib, "xb_expert_gemm", I, [I, I, P, P, P, P, P, I, I, I, I, I, I, I, L, L, I, F, F, P])
-    _sig(lib, "xb_expert_select_gate", I, [I, P, P, P, P, P, I, P, I, I, I, I, I, P, I, F, F, P, P])
+    _sig(lib, "xb_expert_select_gate", I, [I, P, P, P, P, P, I, P, I, I, I, I, I, I, P, P, I, F, F, P, P])
     _sig(lib, "xb_expert_gemm_mma", I, [I, P, P, P, P, P, I, I, I, I, I, I, I, L, L, I, F, F, P])
     _sig(lib, "xb_expert_gather", I, [I, P, P, P, P, I, I, I, I, P])
-    _sig(lib, "xb_expert_combine", I, [I, P, P, P, I, I, I, P, P, P])
-    _sig(lib, "xb_expert_router", I, [I, P, P, P, P, P, P, I, I, I, I, I, I, I, I, P])
+    _sig(lib, "xb_expert_combine", I, [I, P, P, P, I, I, I, P, P, P, P])
+    _sig(lib, "xb_expert_router", I, [I, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, F, F, P])
     _sig(lib, "xb_attn_decode_tc", I, [P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, F, F, F, I, I, I, I, P, I, P, P])

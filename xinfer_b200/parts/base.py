@@ -186,6 +186,10 @@ class Part:
     def load(self, store: WeightStore) -> None:
         pass
 
+    def children(self) -> Sequence["Part"]:
+        """Parts that this one is made of and that hold weights of their own."""
+        return ()
+
 
 class Mixer(Part):
     """Mixes information across the tokens of a request.
@@ -196,7 +200,14 @@ class Mixer(Part):
     ``[T, hidden]``; it must write this step's keys/values (or state) before reading them, and it
     must give the same result however the request's tokens were cut into steps.
     ``writes_cache`` False means this run reads pages another run wrote.
+
+    A mixer that may read the residual stream itself and whose first kernel can form the sum that waits for it says so
+    with ``takes_stream``: the executor then calls ``forward_stream(x, addend, ctx, cache, state, writes_cache)``, which
+    returns the result and the stream after the addition (possibly another tensor), for an addend that
+    ``accepts_addend`` takes.
     """
+
+    takes_stream: bool = False
 
     def cache_need(self) -> Optional[PagedCacheNeed]:
         return None

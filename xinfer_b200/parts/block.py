@@ -9,7 +9,8 @@ reference wires its one arrangement by hand, ``x + mixer(norm(x))`` then ``x + m
 Here an addition is carried out when its sum is next read.  Where a norm reads it, the norm
 kernel forms the sum in float32, stores it and norms it in one pass - also across the block
 boundary: the last addition of a block waits in the ``Stream`` that the next block (or the
-decoder's final norm) receives.  Where a mixer or a feed-forward runs next, an addition kernel
+decoder's final norm) receives.  A mixer whose first kernel can form the sum (``Mixer.takes_stream``) does
+so where it reads the stream itself.  Where a mixer or a feed-forward runs next, an addition kernel
 runs first (for every waiting addition: the part may reuse the buffer an addend lives in).
 The pre-norm block therefore launches exactly the kernels a hand-written one would.
 """
@@ -219,10 +220,17 @@ class Block:
                 if tracing.ENABLED:
                     tracing.pop()
             else:
+                # a mixer that reads the stream itself may form the last waiting sum in its first kernel
+                whole = o.op == "mixer" and o.src == "x" and part.takes_stream
+                last = None
+                if whole and waiting.get("x") and part.accepts_addend(waiting["x"][-1]):
+                    last = waiting["x"].pop()
                 settle_all()
                 if tracing.ENABLED:
                     tracing.push(o.op + ":" + part.kind)
-                if o.op == "mixer":
+                if whole:
+                    out, vals["x"] = part.forward_stream(vals["x"], last, ctx, cache, state, writes_cache)
+                elif o.op == "mixer":
                     out = part.forward(vals[o.src], ctx, cache, state, writes_cache)
                 else:
                     out = part.forward(vals[o.src], ctx)

@@ -30,3 +30,13 @@ def linear(out: torch.Tensor, x: torch.Tensor, weight: torch.Tensor, err: Option
         return out
     kernels.gemm_plain(out, x, weight)
     return out
+
+
+def stack_rows(matrices, multiple: int = 8) -> torch.Tensor:
+    """Matrices that read the same input as one, below each other, with rows of zeros up to a multiple of ``multiple``:
+    the rows of the product then start on 16-byte boundaries in either type."""
+    rows = sum(m.shape[0] for m in matrices)
+    pad = -rows % multiple
+    if pad:
+        matrices = list(matrices) + [torch.zeros((pad, matrices[0].shape[1]), dtype=matrices[0].dtype, device=matrices[0].device)]
+    return torch.cat(matrices, dim=0).contiguous()

@@ -47,6 +47,10 @@ class ParallelMixer(Mixer):
             out += [WeightSpec(prefix + n, (spec.hidden,), "norm") for n in spec.out_norms]
         return out
 
+    def children(self):
+        # with one output product for both sides the combined matrix is this part's, else every side has its own
+        return (self.left, self.right) if self.spec.out_norms is not None else ()
+
     def load(self, store) -> None:
         self.left.load(store)
         self.right.load(store)

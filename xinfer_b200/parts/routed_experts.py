@@ -1,17 +1,19 @@
 """Mixture of small gated experts chosen by a learned router, with an optional expert that every token runs.
 
-    scores   s = sigmoid(W_router h)                     float32
+    scores   s = sigmoid(W_router h), or softmax(W_router h) over all experts       float32
     choice   on s + correction, among the experts of the ``keep`` best of ``groups`` groups of neighbours
              (a group's score: the sum of its ``group_best`` largest choice scores); the ``top`` largest win
-    weights  the chosen experts' plain scores s (optionally divided by their sum)
+    weights  the chosen experts' plain scores s (optionally divided by their sum), times a constant
     expert   W_down_e ( act(W_gate_e h) * f(W_up_e h) ),  no biases; ``act`` by the spec (``kernels.ACTIVATIONS``)
-    out      = sum over the token's experts of weight * expert  (+ shared(h))
+    out      = sum over the token's experts of weight * expert  (+ shared(h), optionally times sigmoid(w_g . h))
 
 The router kernel leaves the step's choices and weights on the device, a row per token; from there the forms of
 the table-driven experts (``parts/table_experts.py``) are reused with that table in place of one over token ids:
 
 * few tokens in bfloat16 (a decode step): ONE dense product with the gate/up matrices stacked, a kernel that keeps a
-  token's own experts (times their weights) and zeroes the others, ONE product with the down matrices side by side;
+  token's own experts (times their weights) and zeroes the others, ONE product with the down matrices side by side; a
+  shared expert with a gate and the experts' own activation takes part in both products as one more block of rows
+  (columns) with the gate as its weight;
 * otherwise: the (token, choice) pairs are grouped by expert on the device, two grouped products run (gate/up with
   the activation applied in the same kernel, then down), and a last kernel sums a token's experts in the order of
   its choices, each times its weight, onto the shared expert's result;
@@ -57,11 +59,19 @@ class RoutedExperts(FeedForward):
         if spec.top > spec.keep * (spec.experts // spec.groups):
             raise ValueError(f"{spec.keep} groups of {spec.experts // spec.groups} experts cannot give a token {spec.top}")
         kernels.activation_args(spec.activation, spec.act_params)
+        if spec.score not in ("sigmoid", "softmax"):
+            raise ValueError(f"a router scores by sigmoid or softmax, not '{spec.score}'")
+        if spec.shared_gate is not None and spec.shared is None:
+            raise ValueError("a gate on the shared expert needs a shared expert")
         self.shared = None
         if spec.shared is not None:
             self.shared = build_part("feed_forward", spec.shared, prefix + "shared.", dtype, device)
             self.shared.scratch = "experts.shared"
-        self.w_gate_up = self.w_down = self.w_router = self.correction = None
+        # the shared expert's matrices lie behind the experts' own: few tokens run both in the same two products
+        self.together = (spec.shared_gate is not None and dtype == torch.bfloat16 and spec.shared.kind == "swiglu"
+                         and spec.shared.bias_suffix is None and spec.shared.activation == spec.activation
+                         and tuple(spec.shared.act_params) == tuple(spec.act_params))
+        self.w_gate_up = self.w_down = self.w_router = self.correction = self.w_gate_up_all = None
 
     @classmethod
     def weight_specs(cls, spec: RoutedExpertsSpec, prefix: str) -> List[WeightSpec]:
@@ -76,7 +86,12 @@ class RoutedExperts(FeedForward):
             out.append(WeightSpec(prefix + "correction", (spec.experts,), "around_zero"))
         if spec.shared is not None:
             out += part_class("feed_forward", spec.shared.kind).weight_specs(spec.shared, prefix + "shared.")
+        if spec.shared_gate is not None:
+            out.append(WeightSpec(prefix + spec.shared_gate, (1, spec.hidden), "unit"))
         return out
+
+    def children(self):
+        return () if self.shared is None or self.together else (self.shared,)
 
     def load(self, store) -> None:
         s, p = self.spec, self.prefix
@@ -86,14 +101,24 @@ class RoutedExperts(FeedForward):
             gu.append(torch.cat([store.get(q + "gate", self.device, self.dtype, operand=True),
                                  store.get(q + "up", self.device, self.dtype, operand=True)], dim=0))
             dn.append(store.get(q + "down", self.device, self.dtype, operand=True))
-        self.w_gate_up = torch.stack(gu).contiguous()      # [experts, 2 ff, hidden]
-        self.w_down = torch.cat(dn, dim=1).contiguous()    # [hidden, experts * ff]: side by side along K
-        # the router works in float32 whatever the engine's type
-        self.w_router = store.get(p + "router", self.device, torch.float32).float().contiguous()
-        if s.correction:
-            self.correction = store.get(p + "correction", self.device, torch.float32).float().contiguous()
         if self.shared is not None:
             self.shared.load(store)
+        if self.together:
+            gu.append(self.shared.w_gate_up)
+            dn.append(self.shared.w_down)
+        rows = s.experts * 2 * s.intermediate
+        self.w_gate_up_all = torch.cat(gu, dim=0).contiguous()
+        self.w_gate_up = self.w_gate_up_all[:rows].view(s.experts, 2 * s.intermediate, s.hidden)
+        self.w_down = torch.cat(dn, dim=1).contiguous()    # [hidden, experts * ff (+ shared ff)]: side by side along K
+        if self.together:
+            self.shared.w_gate_up = self.w_gate_up_all[rows:]       # (the same rows, held once)
+        # the router works in float32 whatever the engine's type; the shared expert's gate is one more row of it
+        router = [store.get(p + "router", self.device, torch.float32).float()]
+        if s.shared_gate is not None:
+            router.append(store.get(p + s.shared_gate, self.device, torch.float32).float())
+        self.w_router = torch.cat(router, dim=0).contiguous()
+        if s.correction:
+            self.correction = store.get(p + "correction", self.device, torch.float32).float().contiguous()
 
     def forward(self, x, ctx: StepContext):
         s = self.spec
@@ -101,16 +126,21 @@ class RoutedExperts(FeedForward):
         ws = ctx.workspace
         choice = ws.get("experts.choice", (T, s.top), torch.int32)
         weight = ws.get("experts.weight", (T, s.top), torch.float32)
+        gate = ws.get("experts.gate", (T,), torch.float32) if s.shared_gate is not None else None
         kernels.expert_router(choice, weight, x, self.w_router, self.correction, ctx.req_of_token, s.top, s.groups, s.keep,
-                              s.group_best, s.renormalize)
-        base = self.shared.forward(x, ctx) if self.shared is not None else None
+                              s.group_best, s.renormalize, softmax=s.score == "softmax", renormalize_eps=s.renormalize_eps,
+                              weight_scale=s.weight_scale, gate=gate)
+        few = self.dtype == torch.bfloat16 and T <= DENSE_MAX_TOKENS and (gate is None or self.together)
+        base = self.shared.forward(x, ctx) if self.shared is not None and not (few and self.together) else None
         out = ws.get("experts.out", (T, s.hidden), ctx.branch_dtype or self.dtype)
-        if self.dtype == torch.bfloat16 and T <= DENSE_MAX_TOKENS:
-            gu = ws.get("experts.gu_all", (T, s.experts * 2 * s.intermediate), self.dtype)
-            linear(gu, x, self.w_gate_up.view(s.experts * 2 * s.intermediate, s.hidden), ctx.err)
-            act = ws.get("experts.act_all", (T, s.experts * s.intermediate), self.dtype)
+        if few:
+            more = s.shared.intermediate if self.together else 0
+            gu = ws.get("experts.gu_all", (T, self.w_gate_up_all.shape[0]), self.dtype)
+            linear(gu, x, self.w_gate_up_all, ctx.err)
+            act = ws.get("experts.act_all", (T, s.experts * s.intermediate + more), self.dtype)
             kernels.expert_select_gate(act, gu, choice, None, None, ctx.req_of_token, s.top, s.experts, ctx.err,
-                                       weights=weight, activation=s.activation, params=s.act_params)
+                                       weights=weight, activation=s.activation, params=s.act_params, dense=more,
+                                       dense_weight=gate)
             linear(out, act, self.w_down, ctx.err)
             if base is not None:
                 kernels.add(out, out, base)
@@ -149,7 +179,7 @@ class RoutedExperts(FeedForward):
             kernels.expert_gemm(act, x, self.w_gate_up, offsets, perm, True, s.top, True, activation=s.activation,
                                 params=s.act_params)
             kernels.expert_gemm(y, act, self.w_down, offsets, perm, False, s.top, False, side_by_side=True)
-        kernels.expert_combine(out, y, inv, s.top, weights=weight, base=base)
+        kernels.expert_combine(out, y, inv, s.top, weights=weight, base=base, base_gate=gate)
         return out
 
 
