@@ -204,3 +204,52 @@ def replay_in_process(runner, steps: List[dict]) -> Dict[int, np.ndarray]:
                 runner.close_request(slots.pop(rid))
     assert not slots, "every request of a trace must end"
     return out
+
+
+def row_error(got, want) -> float:
+    """Root mean square over the vocabulary of the difference, its mean taken off."""
+    d = got.astype(np.float64) - want
+    d = d - d.mean()
+    return float(np.sqrt((d * d).mean()))
+
+
+def replay_with_routes(runner, steps: List[dict], moe_runs: Sequence[int]):
+    """``replay_in_process`` with every router call's choices kept: returns the logits per step and, per request id
+    and layer run (``moe_runs``: the runs that have a router, in order), the experts chosen at every position of the
+    request."""
+    from xinfer_b200 import kernels
+    from xinfer_b200.engine.runner import StepInput
+    calls, orig = [], kernels.expert_router
+
+    def spy(choice, weight, *a, **kw):
+        orig(choice, weight, *a, **kw)
+        calls.append(choice.clone())
+
+    slots, routes, out = {}, {}, {}
+    kernels.expert_router = spy
+    try:
+        for s in steps:
+            calls.clear()
+            entries = []
+            for e in s["entries"]:
+                if e["id"] not in slots:
+                    slots[e["id"]] = runner.open_request()
+                entries.append(StepInput(slots[e["id"]], e["tokens"], e.get("want", [])))
+            logits = runner.step(entries)
+            runner.check_errors()
+            if logits.shape[0]:
+                out[s["step"]] = logits.float().cpu().numpy().copy()
+            assert len(calls) == len(moe_runs)
+            chosen = [c.cpu() for c in calls]
+            row = 0
+            for e in s["entries"]:          # the step's rows are its entries' tokens in order
+                n = len(e["tokens"])
+                for run, c in zip(moe_runs, chosen):
+                    routes.setdefault(e["id"], {}).setdefault(run, []).append(c[row:row + n])
+                row += n
+            for rid in s.get("end", []):
+                runner.close_request(slots.pop(rid))
+    finally:
+        kernels.expert_router = orig
+    assert not slots
+    return out, {rid: {run: torch.cat(parts) for run, parts in per.items()} for rid, per in routes.items()}

@@ -10,7 +10,7 @@ import torch
 
 import plain_mikutar as plain
 from mikutar_models import TINY_M, make_folder, prompts
-from helpers import build_all_modes, replay_in_process, run_trace
+from helpers import build_all_modes, replay_with_routes, row_error, run_trace
 
 pytestmark = pytest.mark.gpu
 
@@ -393,13 +393,6 @@ def test_the_cap_bounds_a_score_and_the_slope_orders_equal_keys(dtype, tiled):
 LENGTHS = {"M1": [70, 45, 130, 33], "M2": [97, 41, 260, 150], "M3": [170, 1, 75, 58], "M4": [90, 2, 51, 140]}
 
 
-def _row_error(got, want):
-    """Root mean square over the vocabulary of the difference, its mean taken off."""
-    d = got.astype(np.float64) - want
-    d = d - d.mean()
-    return float(np.sqrt((d * d).mean()))
-
-
 def _tolerance(dtype, ref, cfg=None, w=None, p=None):
     """float32: a small share of the logits' spread (the engine's float32 against float64).  bfloat16: three
     times what rounding alone causes - the largest row error of the plain run that rounds activations to
@@ -408,7 +401,7 @@ def _tolerance(dtype, ref, cfg=None, w=None, p=None):
     if dtype == "float32":
         return 3e-5 * spread
     rounded = plain.forward(cfg, w, p, round_to=torch.bfloat16).numpy()
-    return max(3.0 * max(_row_error(rounded[i], ref[i]) for i in range(len(p))), 1e-3 * spread)
+    return max(3.0 * max(row_error(rounded[i], ref[i]) for i in range(len(p))), 1e-3 * spread)
 
 
 def _store(dtype):
@@ -431,55 +424,13 @@ def test_every_way_of_cutting_gives_the_plain_logits_in_float32_through_the_repl
         got = out[step]
         assert got.shape[0] == len(rows)
         for r, ((mode, i), pos) in enumerate(rows):
-            e = _row_error(got[r], ref[i][pos])
+            e = row_error(got[r], ref[i][pos])
             assert e <= tol[i], (f"{name} {mode}: request {i} position {pos} (step {step}) differs by {e:.3g} "
                                  f"> {tol[i]:.3g}: the first wrong token of this mode")
             seen.setdefault((mode, i), set()).add(pos)
     for mode in ("whole", "tail", "portions", "mixed"):
         for i, p in enumerate(ps):
             assert sorted(seen[(mode, i)]) == list(range(len(p))), (mode, i)
-
-
-def _replay_with_routes(runner, steps, moe_runs):
-    """``replay_in_process`` with every router call's choices kept: returns the logits per step and, per request id
-    and layer run, the experts chosen at every position of the request."""
-    from xinfer_b200 import kernels
-    from xinfer_b200.engine.runner import StepInput
-    calls, orig = [], kernels.expert_router
-
-    def spy(choice, weight, *a, **kw):
-        orig(choice, weight, *a, **kw)
-        calls.append(choice.clone())
-
-    slots, at, routes, out = {}, {}, {}, {}
-    kernels.expert_router = spy
-    try:
-        for s in steps:
-            calls.clear()
-            entries = []
-            for e in s["entries"]:
-                if e["id"] not in slots:
-                    slots[e["id"]] = runner.open_request()
-                    at[e["id"]] = 0
-                entries.append(StepInput(slots[e["id"]], e["tokens"], e.get("want", [])))
-            logits = runner.step(entries)
-            runner.check_errors()
-            if logits.shape[0]:
-                out[s["step"]] = logits.float().cpu().numpy().copy()
-            assert len(calls) == len(moe_runs)
-            chosen = [c.cpu() for c in calls]
-            row = 0
-            for e in s["entries"]:          # the step's rows are its entries' tokens in order
-                n = len(e["tokens"])
-                for run, c in zip(moe_runs, chosen):
-                    routes.setdefault(e["id"], {}).setdefault(run, []).append(c[row:row + n])
-                row += n
-            for rid in s.get("end", []):
-                runner.close_request(slots.pop(rid))
-    finally:
-        kernels.expert_router = orig
-    assert not slots
-    return out, {rid: {run: torch.cat(parts) for run, parts in per.items()} for rid, per in routes.items()}
 
 
 def _check_trace(name, dtype, runner, tb, ps, cfg, w):
@@ -489,7 +440,7 @@ def _check_trace(name, dtype, runner, tb, ps, cfg, w):
     the plain run (in float32 nothing is close: the slack is a rounding error's)."""
     order = plain.layer_order(cfg)
     moe_runs = [run for run, (i, _) in enumerate(order) if (cfg["layers"][i].get("mlp") or {}).get("kind") == "moe"]
-    out, routes = _replay_with_routes(runner, tb.steps, moe_runs)
+    out, routes = replay_with_routes(runner, tb.steps, moe_runs)
     slack = 1e-5 if dtype == "float32" else 0.05
     ref, tol = {}, {}         # per request id of the trace: the plain logits along the engine's routes
 
@@ -508,7 +459,7 @@ def _check_trace(name, dtype, runner, tb, ps, cfg, w):
         rid_of_row = [e["id"] for e in tb.steps[step]["entries"] for _ in e["want"]]
         for r, ((mode, i), pos) in enumerate(rows):
             want, t = plain_of(rid_of_row[r], i)
-            e = _row_error(got[r], want[pos])
+            e = row_error(got[r], want[pos])
             worst[mode] = max(worst.get(mode, 0.0), e / t)
             assert e <= t, (f"{name} {dtype} {mode}: request {i} position {pos} (step {step}) differs by {e:.3g} "
                             f"> {t:.3g}: the first wrong token of this mode")

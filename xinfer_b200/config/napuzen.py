@@ -101,14 +101,12 @@ def _mixer(kind: str, m, wm: str) -> NapuzenMixer:
     if kind == "gla":
         return NapuzenMixer(**sizes, tau=_num(m, "tau", wm, positive=True))
     latent = dict(scale=_num(m, "scale", wm), kv_rank=_int(m, "kv_rank", wm))
-    if kind == "latent_attention":
+    if kind == LATENT_TYPES[0]:
         rot_dim = _int(m, "rot_dim", wm, least=2)
         return NapuzenMixer(**sizes, **latent, q_rank=_int(m, "q_rank", wm), rot_dim=rot_dim,
                             rot=_rot(_get(m, "rot", wm), wm + "rot.", rot_dim))
-    if kind == "latent_attention_2":
-        kv_from = _int(m, "kv_from", wm, least=0) if m.get("kv_from") is not None else None
-        return NapuzenMixer(**sizes, **latent, window=_int(_get(m, "mask", wm), "size", wm + "mask."), kv_from=kv_from)
-    raise ConfigError(f"config key '{wm[:-6]}type' is '{kind}'; known: gla, {', '.join(LATENT_TYPES)}")
+    kv_from = _int(m, "kv_from", wm, least=0) if m.get("kv_from") is not None else None
+    return NapuzenMixer(**sizes, **latent, window=_int(_get(m, "mask", wm), "size", wm + "mask."), kv_from=kv_from)
 
 
 def _mlp(f, wf: str) -> NapuzenMlp:
@@ -150,6 +148,8 @@ class NapuzenConfig:
         for i, layer in enumerate(layers):
             w = f"layers[{i}]."
             kind = _get(layer, "type", w)
+            if kind != "gla" and kind not in LATENT_TYPES:
+                raise ConfigError(f"config key '{w}type' is '{kind}'; known: gla, {', '.join(LATENT_TYPES)}")
             mixer = _mixer(kind, _get(layer, "mixer", w), w + "mixer.")
             mlp = _mlp(layer["mlp"], w + "mlp.") if layer.get("mlp") is not None else None
             out.append(NapuzenLayer(kind, mixer, mlp))

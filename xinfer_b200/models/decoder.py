@@ -76,19 +76,21 @@ class DecoderModel:
 
     def weight_bytes(self) -> int:
         seen, total = set(), 0
-        def visit(obj):
+        def count(t):
             nonlocal total
+            mem = t.untyped_storage()       # parts may hold several views of one matrix
+            if mem.data_ptr() not in seen:
+                seen.add(mem.data_ptr())
+                total += mem.nbytes()
+        def visit(obj):
             for v in vars(obj).values():
-                if isinstance(v, torch.Tensor) and v.data_ptr() not in seen:
-                    seen.add(v.data_ptr())
-                    total += v.numel() * v.element_size()
+                if isinstance(v, torch.Tensor):
+                    count(v)
         visit(self)
         visit(self.final_norm)
         for b in self.blocks:
             for t in b.gains.values():
-                if t.data_ptr() not in seen:
-                    seen.add(t.data_ptr())
-                    total += t.numel() * t.element_size()
+                count(t)
             for part in b.all_parts():
                 stack = [part]
                 while stack:
