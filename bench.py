@@ -10,6 +10,7 @@
     python bench.py --compare dufitar [--size 1k|4k]        # the Dufitar design beside Qwen3 at equal layer sizes
     python bench.py --compare gulipel [--size 1k|4k]        # the Gulipel design beside Tidarax at equal layer sizes
     python bench.py --compare mikutar [--size 1k|4k]        # the Mikutar design beside Dufitar at equal layer sizes
+    python bench.py --compare napuzen [--size 1k|4k]        # the Napuzen design beside Dufitar and Gulipel at equal layer sizes
 
 Prints ONE JSON line.  ``value`` is decoded tokens per second at batch 8 and the context length
 of the configuration (a "step" is one decode step of the whole batch), timed on the device with
@@ -298,6 +299,33 @@ def mikutar_config(z: dict, layers: int, vocab: int, loop: bool = False) -> dict
     return cfg
 
 
+# --compare napuzen: linear attention / dense, latent attention without positions / experts, linear attention / dense,
+# latent attention with a rotated part / experts; the linear attention with as many heads as the other designs' attention,
+# latents and experts of the sizes above, windows wider than the benchmark's context, queries through a latent of three
+# times the cached one's size.
+def napuzen_config(z: dict, lat: dict, layers: int, vocab: int) -> dict:
+    H, d, r = z["heads"], z["head_dim"], lat["kv_rank"]
+    gla = dict(type="gla", mixer=dict(heads=H, dim=d, vdim=d, tau=8.0))
+    rot = dict(dims=lat["rot_dim"], base=100000.0, scaling=dict(factor=4.0, original=8192, fast=16.0, slow=2.0))
+    latent = dict(type="latent_attention", mixer=dict(heads=H, dim=d, rot_dim=lat["rot_dim"], vdim=d, q_rank=3 * r, kv_rank=r,
+                                                      scale=(d + lat["rot_dim"]) ** -0.5, rot=rot))
+
+    def latent2(kv_from=None):
+        m = dict(heads=H, dim=d, vdim=d, kv_rank=r, scale=d ** -0.5, mask=dict(size=COMPARE_WINDOW))
+        if kv_from is not None:
+            m["kv_from"] = kv_from
+        return dict(type="latent_attention_2", mixer=m)
+    dense = dict(kind="dense", ff=z["intermediate"], limit=7.0)
+    moe = dict(kind="moe", expert=dict(ff=z["expert_ff"]), shared=dict(ff=z["expert_ff"]),
+               router=dict(experts=z["experts"], top=z["top"], scale=1.5))
+    out = []
+    for i in range(layers):
+        mixer = gla if i % 2 == 0 else (latent if i % 4 == 3 else latent2(i - 4 if i % 8 == 5 else None))
+        out.append(dict(mixer, mlp=moe if i % 2 else dense))
+    return dict(architecture="Napuzen", vocab=vocab, width=z["hidden"], norm=dict(eps=1e-6), canon=dict(taps=4), logit_scale=0.8,
+                layers=out)
+
+
 def compare(args) -> int:
     """Prefill and decode throughput of a model of the named design and of a Qwen3 model of the same layer sizes
     (random weights, `--layers` layers each, default 4), then the design's kernels one by one beside their like
@@ -316,6 +344,9 @@ def compare(args) -> int:
     elif args.compare == "mikutar":     # its closest model is the other one with gated window attention and a float32 stream
         models = {"Mikutar": mikutar_config(z, L, V), "Mikutar, first layers twice": mikutar_config(z, L, V, loop=True),
                   "Dufitar": dufitar_config(z, LATENT_SIZES[args.size], L, V)}
+    elif args.compare == "napuzen":     # latent attention as in Dufitar, a recurrence with a matrix state as in Gulipel
+        models = {"Napuzen": napuzen_config(z, LATENT_SIZES[args.size], L, V), "Dufitar": dufitar_config(z, LATENT_SIZES[args.size], L, V),
+                  "Gulipel": gulipel_config(z, L, V, ctx_len + 128)}
     elif args.compare == "tidarax":
         models = {"Tidarax": tidarax_config(z, L, V), "Qwen3": qwen3}
     else:
@@ -369,6 +400,11 @@ def compare(args) -> int:
         records = measure.mikutar_kernels(hidden=z["hidden"], heads=z["heads"], kv_heads=z["kv_heads"], head_dim=z["head_dim"],
                                           intermediate=z["intermediate"], experts=z["experts"], expert_ff=z["expert_ff"],
                                           top=z["top"], hbm_gbs=pk["hbm_gbs"], peak_tflops=pk["bf16_tflops"])
+    elif args.compare == "napuzen":
+        lat = LATENT_SIZES[args.size]
+        records = measure.napuzen_kernels(hidden=z["hidden"], heads=z["heads"], head_dim=z["head_dim"], kv_rank=lat["kv_rank"],
+                                          rot_dim=lat["rot_dim"], q_rank=3 * lat["kv_rank"], experts=z["experts"],
+                                          expert_ff=z["expert_ff"], top=z["top"], hbm_gbs=pk["hbm_gbs"], peak_tflops=pk["bf16_tflops"])
     elif args.compare == "gulipel":
         records = measure.gulipel_kernels(hidden=z["hidden"], heads=z["heads"], kv_heads=z["kv_heads"], head_dim=z["head_dim"],
                                           intermediate=z["intermediate"], hbm_gbs=pk["hbm_gbs"], **gulipel_sizes(z))
@@ -410,9 +446,9 @@ def main() -> int:
                     help="with --kernels: the attention kernels alone at this head layout, over short and long contexts")
     ap.add_argument("--case", default="", metavar="decode:BATCHxCONTEXT | prefill:CACHED+NEW",
                     help="with --kernels --attn: this one case instead of the standard ones")
-    ap.add_argument("--compare", default="", choices=["", "tidarax", "dufitar", "gulipel", "mikutar"],
+    ap.add_argument("--compare", default="", choices=["", "tidarax", "dufitar", "gulipel", "mikutar", "napuzen"],
                     help="instead of the step benchmark: prefill and decode throughput of this design beside its closest model "
-                         "(Qwen3; for gulipel, Tidarax) at equal layer sizes, and its kernels beside their like kernels; one JSON line each")
+                         "(Qwen3; for gulipel, Tidarax; for mikutar, Dufitar; for napuzen, Dufitar and Gulipel) at equal layer sizes, and its kernels beside their like kernels; one JSON line each")
     ap.add_argument("--size", default="4k", choices=sorted(COMPARE_SIZES), help="layer sizes of --compare")
     ap.add_argument("--kernels", action="store_true",
                     help="instead of the step benchmark, time single kernels at serving sizes: one JSON line each")

@@ -827,3 +827,168 @@ def mikutar_kernels(*, hidden: int = 4096, heads: int = 32, kv_heads: int = 8, h
     if int(err):
         raise RuntimeError("a kernel reported an error: " + kernels.describe_error(int(err)))
     return out
+
+
+def napuzen_kernels(*, hidden: int = 4096, heads: int = 32, head_dim: int = 128, kv_rank: int = 512, rot_dim: int = 64,
+                    q_rank: int = 1536, rank: int = 16, conv: int = 4, experts: int = 8, expert_ff: int = 3072, top: int = 2,
+                    tokens: int = 2048, decode: Sequence[int] = (8, 4096), page_size: int = 16, hbm_gbs: float = 0.0,
+                    peak_tflops: float = 0.0, device="cuda:0") -> List[Dict]:
+    """One record per kernel of the Napuzen path: time, bytes and the share of its floor (the bytes that must cross
+    memory at the measured copy rate; for the scan also its arithmetic at the nominal FMA rate, for the attention its
+    products at the measured matrix-product peak), each followed by the like kernel of the design it is closest to,
+    measured the same way ("like: ...")."""
+    from .parts import latent_attention as la
+    out: List[Dict] = []
+    err = torch.zeros(1, dtype=torch.int32, device=device)
+    sets = 4
+    f32 = lambda *shape: torch.randn(*shape, device=device)
+    bf = lambda *shape: torch.randn(*shape, device=device).bfloat16()
+    i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=device)
+
+    def record(name, nbytes, run, flops=0.0, tensor_flops=0.0, n=sets, **more):
+        us = _graph_time_us(lambda: [run(i) for i in range(n)], n)
+        floor_us = nbytes / (hbm_gbs or 6650.0) / 1e3
+        if flops:
+            floor_us = max(floor_us, flops / FP32_FMA_TFLOPS_NOMINAL / 1e6)
+        if tensor_flops:
+            floor_us = max(floor_us, tensor_flops / (peak_tflops or 1590.0) / 1e6)
+        out.append(dict({"kernel": name, "bytes": nbytes, "us": round(us, 1), "gbs": round(nbytes / us / 1e3, 1),
+                         "floor_us": round(floor_us, 2), "frac_of_floor": round(floor_us / us, 3)}, **more))
+
+    B, context = decode
+    steps = (("a prompt", tokens, i32([0, tokens]), i32([0]), torch.zeros(tokens, dtype=torch.int32, device=device), 1),
+             ("single tokens", B, i32(list(range(B + 1))), i32(list(range(B))), i32(list(range(B))), B))
+    H, d, C = heads, head_dim, hidden
+    w, w2, gain = f32(C), f32(C), f32(C)
+
+    # the stream: branch norm, sum and the convolution behind it; branch norm, sum and the hand-over to the feed-forward
+    for what, T, qs, sl, rq, ne in steps:
+        xs, ss, bs = [f32(T, C) for _ in range(sets)], [f32(T, C) for _ in range(sets)], [f32(T, C) for _ in range(sets)]
+        hs = [torch.empty(T, C, dtype=torch.bfloat16, device=device) for _ in range(sets)]
+        states = [torch.zeros(ne, conv - 1, C, device=device) for _ in range(sets)]
+        taps = f32(C, conv)
+        record(f"normed branch + float32 sum + convolution of {conv} taps, {what}", T * C * 14 + 2 * ne * (conv - 1) * C * 4,
+               lambda i: kernels.stream_conv(hs[i], xs[i], taps, states[i], rq, qs, sl, ne, branch=bs[i], branch_weight=w,
+                                             branch_eps=1e-6, sum_out=ss[i], single=T == B), tokens=T)
+        record(f"normed branch + float32 sum, handed over in bfloat16, {what}", T * C * 14,
+               lambda i: kernels.rms_chain(hs[i], xs[i], None, 0.0, err, branch=bs[i], branch_weight=w, branch_eps=1e-6, sum_out=xs[i]),
+               tokens=T)
+        record(f"like: Gulipel normed branch x learned scale + float32 sum + norm, {what}", T * C * 14,
+               lambda i: kernels.rms_chain(hs[i], xs[i], w, 1e-6, err, branch=bs[i], branch_weight=w2, branch_eps=1e-6, gain=gain,
+                                           sum_out=xs[i]), tokens=T)
+        del xs, ss, bs, hs, states
+
+    # gated linear attention beside the gated delta rule
+    qk = H * d
+    for what, T, qs, sl, rq, ne in steps:
+        projs = [f32(T, 4 * qk + rank) for _ in range(sets)]
+        alphas = [torch.rand(T, qk, device=device) for _ in range(sets)]
+        os_ = [torch.empty(T, qk, device=device) for _ in range(sets)]
+        gated = [torch.empty(T, qk, dtype=torch.bfloat16, device=device) for _ in range(sets)]
+        states = [torch.zeros(ne, H, d, d, device=device) for _ in range(sets)]
+        wd, bd, nw = f32(qk, rank), f32(qk), f32(d)
+        record(f"decay from the low-rank map, {what}", T * (qk + rank) * 4 + qk * (rank + 1) * 4,
+               lambda i: kernels.low_rank_decay(alphas[i], projs[i][:, 4 * qk:], wd, bd, 8.0), tokens=T)
+        record(f"linear attention scan, {what}", T * 5 * qk * 4 + 2 * ne * qk * d * 4,
+               lambda i: kernels.linear_scan(os_[i], projs[i], alphas[i], states[i], qs, sl, ne, H, d, d, d ** -0.5),
+               flops=6.0 * T * qk * d, tokens=T, heads=H, dim=d)
+        record(f"norm per head + SiLU gate, {what}", T * qk * 10,
+               lambda i: kernels.gated_head_norm(gated[i], os_[i], projs[i], 3 * qk, nw, d, 1e-6, gate_after=True, silu_gate=True),
+               tokens=T)
+        qkvs, betas = [f32(T, 3 * qk) for _ in range(sets)], [f32(T, 3 * qk + H) for _ in range(sets)]
+        ags = [f32(T, 2 * qk) for _ in range(sets)]
+        alog = f32(H)
+        record(f"like: Gulipel gated delta rule, {what}", T * (6 * qk + H) * 4 + 2 * ne * qk * d * 4,
+               lambda i: kernels.delta_rule(os_[i], qkvs[i], betas[i], 3 * qk, ags[i], bd, alog, states[i], qs, sl, ne, H, H, d, d),
+               flops=8.0 * T * qk * d, tokens=T, heads=H, dim=d)
+        record(f"like: Gulipel norm per head + sigmoid gate, {what}", T * qk * 10,
+               lambda i: kernels.gated_head_norm(gated[i], os_[i], ags[i], qk, nw, d, 1e-6, gate_after=True), tokens=T)
+        del projs, alphas, os_, gated, states, qkvs, betas, ags
+
+    # attention over cached rows without a rotated part (rows of the latent alone) and with one, beside Dufitar's with a sink
+    sink = f32(H)
+    for what, entries, single in (("a prompt", [(0, tokens)], False), ("single tokens", [(context - 1, 1)] * B, True)):
+        ctx, table, stride, num_pages = _attention_context(entries, page_size, device)
+        ctx.all_single = single
+        T = ctx.num_tokens
+        pairs = B * context if single else tokens * (tokens + 1) / 2
+        for label, dk, sk in (("latent attention without positions", kv_rank, None), ("latent attention with a rotated part", kv_rank + rot_dim, None),
+                              ("like: Dufitar latent attention with a sink", kv_rank + rot_dim, sink)):
+            n = 4 if single else 1
+            rows = [bf(num_pages, page_size, dk) for _ in range(n)]
+            q, o = bf(T, H, dk) * dk ** -0.5, torch.empty(T, H, kv_rank, dtype=torch.bfloat16, device=device)
+            nbytes = (B * context if single else tokens) * dk * 2 + T * H * (dk + kv_rank) * 2
+            record(f"{label}, {what}", nbytes, lambda i: la.latent_attend(o, q, rows[i], ctx, table, stride, page_size, None, 1.0, sk),
+                   tensor_flops=2.0 * H * (dk + kv_rank) * pairs, n=n, tokens=T)
+            del rows, q, o
+
+    # the rows and queries around it
+    T, r, rd = tokens, kv_rank, rot_dim
+    pages = (T + page_size - 1) // page_size
+    pos = torch.arange(T, dtype=torch.int32, device=device)
+    req = torch.zeros(T, dtype=torch.int32, device=device)
+    tab = torch.randperm(pages, device=device).to(torch.int32)
+    inv = torch.rand(rd // 2, device=device)
+    nw, qw = f32(r), f32(q_rank)
+    lcs = [torch.zeros(pages, page_size, r + rd, dtype=torch.bfloat16, device=device) for _ in range(sets)]
+    projs = [bf(T, q_rank + r + rd) for _ in range(sets)]
+    cqs = [torch.empty(T, q_rank, dtype=torch.bfloat16, device=device) for _ in range(sets)]
+    record("queries' latent norm, latent row norm + rotation + row write", T * 2 * (q_rank + r + rd) * 2,
+           lambda i: kernels.latent_prepare(None, lcs[i], projs[i], 0, q_rank, None, nw, inv, pos, req, tab, pages, 0, d, rd, r, rd,
+                                            1e-6, 1.1, err, query_latent=(cqs[i], 0, qw)), tokens=T)
+    qs_ = [bf(T, H * (d + rd)) for _ in range(sets)]
+    qas = [torch.empty(T, H, r + rd, dtype=torch.bfloat16, device=device) for _ in range(sets)]
+    record("rotation of the queries' rotated parts", T * 2 * H * rd * 2,
+           lambda i: kernels.latent_prepare(qas[i], lcs[i], qs_[i], 0, -1, None, None, inv, pos, req, tab, pages, H, d, rd, r, rd, 1e-6,
+                                            1.1, err), tokens=T)
+    lc2 = [torch.zeros(pages, page_size, r, dtype=torch.bfloat16, device=device) for _ in range(sets)]
+    pr2 = [bf(T, H * d + r + H) for _ in range(sets)]
+    record("latent row norm + row write, no positions", T * 2 * r * 2,
+           lambda i: kernels.latent_prepare(None, lc2[i], pr2[i], 0, H * d, None, nw, None, pos, req, tab, pages, 0, d, 0, r, 0, 1e-6,
+                                            1.0, err), tokens=T)
+    inns = [bf(T, H * d) for _ in range(sets)]
+    record("sigmoid gate of one number per head (in place)", 2 * T * H * d * 2,
+           lambda i: kernels.gate_sigmoid(inns[i], inns[i].view(T, H, d).transpose(0, 1), pr2[i][:, H * d + r:]), tokens=T)
+    pr3 = [bf(T, H * (d + rd) + r + rd) for _ in range(sets)]
+    record("like: Dufitar latent norm + rotation of key part and queries + row write", T * 2 * (H * rd + r + rd) * 2,
+           lambda i: kernels.latent_prepare(qas[i], lcs[i], pr3[i], 0, H * (d + rd), None, nw, inv, pos, req, tab, pages, H, d, rd, r, rd,
+                                            1e-6, 1.0, err), tokens=T)
+    del lcs, projs, cqs, qs_, qas, lc2, pr2, inns, pr3
+
+    # router and experts
+    E, Fi = experts, expert_ff
+    wr = f32(E + 1, C) * C ** -0.5
+    for what, T, qs, sl, rq, ne in steps:
+        hs = [bf(T, C) for _ in range(sets)]
+        choice, weight = torch.zeros(T, top, dtype=torch.int32, device=device), torch.zeros(T, top, device=device)
+        gate = torch.zeros(T, device=device)
+        corr, w_like = f32(E) * 0.3, wr[:E].contiguous()
+        record(f"softmax router with the shared expert's gate, {what}", T * C * 2 + (E + 1) * C * 4,
+               lambda i: kernels.expert_router(choice, weight, hs[i], wr, None, rq, top, renormalize=True, softmax=True,
+                                               renormalize_eps=1e-20, weight_scale=1.5, gate=gate), tokens=T)
+        record(f"like: Mikutar sigmoid router with groups, {what}", T * C * 2 + E * C * 4,
+               lambda i: kernels.expert_router(choice, weight, hs[i], w_like, corr, rq, top, 4, 2, 2), tokens=T)
+        if T == tokens:
+            nrows = T * top
+            offsets, perm, inv_ = i32([0] * (E + 1)), i32([0] * nrows), i32([0] * nrows)
+            kernels.expert_route(offsets, perm, inv_, choice, None, None, rq, T, top, E, err)
+            ys, bases = [f32(nrows, C) for _ in range(sets)], [f32(T, C) for _ in range(sets)]
+            outs = [torch.empty(T, C, device=device) for _ in range(sets)]
+            record(f"experts' weighted sum onto the gated shared expert, {what}", T * C * 4 * (top + 2),
+                   lambda i: kernels.expert_combine(outs[i], ys[i], inv_, top, weights=weight, base=bases[i], base_gate=gate), tokens=T)
+            record(f"like: Mikutar experts' weighted sum onto the shared expert, {what}", T * C * 4 * (top + 2),
+                   lambda i: kernels.expert_combine(outs[i], ys[i], inv_, top, weights=weight, base=bases[i]), tokens=T)
+            del ys, bases, outs
+        else:
+            gus, acts = [bf(T, 2 * (E + 1) * Fi) for _ in range(sets)], [bf(T, (E + 1) * Fi) for _ in range(sets)]
+            record(f"selection and gates of all experts and the shared one, {what}", T * ((top + 1) * 2 + E + 1) * Fi * 2,
+                   lambda i: kernels.expert_select_gate(acts[i], gus[i], choice, None, None, rq, top, E, err, weights=weight, dense=Fi,
+                                                        dense_weight=gate), tokens=T)
+            g2, a2 = [bf(T, 2 * E * Fi) for _ in range(sets)], [bf(T, E * Fi) for _ in range(sets)]
+            record(f"like: Mikutar selection and gates of all experts, {what}", T * (top * 2 + E) * Fi * 2,
+                   lambda i: kernels.expert_select_gate(a2[i], g2[i], choice, None, None, rq, top, E, err, weights=weight,
+                                                        activation="swish_clamp", params=(7.0, 1.702)), tokens=T)
+            del gus, acts, g2, a2
+    if int(err):
+        raise RuntimeError("a kernel reported an error: " + kernels.describe_error(int(err)))
+    return out
