@@ -10,7 +10,7 @@
 //              or s_e / (sum of the chosen s + renorm_eps) where `renorm` is set; times `weight_scale`
 //   gate     = sigmoid(w_g . h), one number per token (a further row of the matrix; absent: none)
 //
-// One block of four warps takes ROUTER_TOKENS consecutive tokens: one, so that a step of few tokens still spreads over
+// One block of four to eight warps (enough for one pass over the rows, where eight are) takes ROUTER_TOKENS consecutive tokens: one, so that a step of few tokens still spreads over
 // the machine (blocks that run on one SM at the same time find the matrix in its L1), or two for steps of thousands
 // of tokens.  First the logits: a warp takes an expert's row of W_r once for the block's tokens, lanes over the
 // channels, four at a time where the rows allow it.  Then the choice: a warp per token.  A token's sums run in an
@@ -20,7 +20,7 @@
 
 #include <math_constants.h>
 
-constexpr int ROUTER_THREADS = 128;
+constexpr int ROUTER_MAX_WARPS = 8;
 
 template <typename T>
 __device__ __forceinline__ void router_load4(const T* p, float (&v)[4]);
@@ -38,7 +38,7 @@ __device__ __forceinline__ void router_load4<__nv_bfloat16>(const __nv_bfloat16*
 }
 
 template <typename T, int ROUTER_TOKENS>
-__global__ void __launch_bounds__(ROUTER_THREADS)
+__global__ void __launch_bounds__(ROUTER_MAX_WARPS * 32)
 expert_router_kernel(int* __restrict__ choice, float* __restrict__ weight, const T* __restrict__ h,
                      const float* __restrict__ w_r, const float* __restrict__ correction,
                      const int* __restrict__ req_of_token, float* __restrict__ gate, int tokens, int E, int K, int top,
@@ -212,8 +212,10 @@ XB_EXPORT int xb_expert_router(int dtype, int* choice, float* weight, const void
     const size_t esz = dtype == XB_F32 ? 4 : 2;
     const int vec4 = (K % 4 == 0 && !((uintptr_t)h & (4 * esz - 1)) && !((uintptr_t)w_r & 15)) ? 1 : 0;
     const unsigned blocks = (unsigned)((tokens + per_block - 1) / per_block);
+    const int rows = experts + (gate != nullptr ? 1 : 0);
+    const int threads = 32 * (rows <= 8 ? 4 : (rows >= 2 * ROUTER_MAX_WARPS ? ROUTER_MAX_WARPS : (rows + 1) / 2));
 #define XB_ROUTER(T, N)                                                                                                   \
-    expert_router_kernel<T, N><<<blocks, ROUTER_THREADS, smem, stream>>>(choice, weight, (const T*)h, w_r, correction,    \
+    expert_router_kernel<T, N><<<blocks, threads, smem, stream>>>(choice, weight, (const T*)h, w_r, correction,    \
                                                                          req_of_token, gate, tokens, experts, K, top,     \
                                                                          groups, keep, group_best, softmax, renorm,       \
                                                                          renorm_eps, weight_scale, vec4)

@@ -474,41 +474,54 @@ __global__ void __launch_bounds__(384, 1) linear_scan_kernel(float* __restrict__
 }
 
 // alpha[t, c] = sigmoid(z)^(1 / tau) = exp(-softplus(-z) / tau),  z = bias[c] + sum_r w[c, r] low[t, r].  low is a
-// column range of wider float32 rows.  A thread per channel and a tile of tokens; r in order for every output.
-constexpr int kDecayTokens = 8, kDecayRanks = 32;
-__global__ void __launch_bounds__(128) low_rank_decay_kernel(float* __restrict__ alpha, const float* __restrict__ low,
-                                                             long long ldl, const float* __restrict__ w,
-                                                             const float* __restrict__ bias, int tokens, int C, int R,
-                                                             float inv_tau) {
-    __shared__ float sl[kDecayRanks][kDecayTokens];
+// column range of wider float32 rows.  A block takes a tile of tokens and 128 channels, a thread one channel of all its
+// tokens; both operands pass through shared memory, so that memory is read in order; r in order for every output.
+constexpr int kDecayTokens = 16, kDecayRanks = 16, kDecayChannels = 128;
+__global__ void __launch_bounds__(kDecayChannels) low_rank_decay_kernel(float* __restrict__ alpha, const float* __restrict__ low,
+                                                                        long long ldl, const float* __restrict__ w,
+                                                                        const float* __restrict__ bias, int tokens, int C, int R,
+                                                                        float inv_tau) {
+    __shared__ __align__(16) float sl[kDecayRanks][kDecayTokens];
+    __shared__ float sw[kDecayRanks][kDecayChannels + 1];
     const int tb = blockIdx.x * kDecayTokens, nt = min(kDecayTokens, tokens - tb);
-    const int c = blockIdx.y * blockDim.x + threadIdx.x;
+    const int c0 = blockIdx.y * kDecayChannels, c = c0 + threadIdx.x;
     float z[kDecayTokens];
     const float b = c < C ? bias[c] : 0.f;
 #pragma unroll
     for (int i = 0; i < kDecayTokens; ++i) z[i] = b;
     for (int r0 = 0; r0 < R; r0 += kDecayRanks) {
-        const int nr = min(kDecayRanks, R - r0);
         if (r0 > 0) __syncthreads();
-        for (int i = threadIdx.x; i < kDecayRanks * kDecayTokens; i += blockDim.x) {
+        for (int i = threadIdx.x; i < kDecayRanks * kDecayTokens; i += kDecayChannels) {
             const int tt = i / kDecayRanks, r = i % kDecayRanks;
-            sl[r][tt] = (tt < nt && r < nr) ? low[(size_t)(tb + tt) * ldl + r0 + r] : 0.f;
+            sl[r][tt] = (tt < nt && r0 + r < R) ? low[(size_t)(tb + tt) * ldl + r0 + r] : 0.f;
+        }
+        for (int i = threadIdx.x; i < kDecayRanks * kDecayChannels; i += kDecayChannels) {
+            const int cc = i / kDecayRanks, r = i % kDecayRanks;
+            sw[r][cc] = (c0 + cc < C && r0 + r < R) ? w[(size_t)(c0 + cc) * R + r0 + r] : 0.f;
         }
         __syncthreads();
-        if (c < C) {
-            const float* wr = w + (size_t)c * R + r0;
-#pragma unroll 8
-            for (int r = 0; r < nr; ++r) {
-                const float wv = wr[r];
 #pragma unroll
-                for (int i = 0; i < kDecayTokens; ++i) z[i] = fmaf(wv, sl[r][i], z[i]);
+        for (int r = 0; r < kDecayRanks; ++r) {
+            const float wv = sw[r][threadIdx.x];
+#pragma unroll
+            for (int i = 0; i < kDecayTokens; i += 4) {
+                const float4 l4 = *reinterpret_cast<const float4*>(&sl[r][i]);
+                z[i] = fmaf(wv, l4.x, z[i]);
+                z[i + 1] = fmaf(wv, l4.y, z[i + 1]);
+                z[i + 2] = fmaf(wv, l4.z, z[i + 2]);
+                z[i + 3] = fmaf(wv, l4.w, z[i + 3]);
             }
         }
     }
     if (c >= C) return;
 #pragma unroll
     for (int i = 0; i < kDecayTokens; ++i)
-        if (i < nt) alpha[(size_t)(tb + i) * C + c] = expf(-softplus_f32(-z[i]) * inv_tau);
+        if (i < nt) {
+            // softplus(-z) without a branch.  What enters the sum's logarithm lies in (1, 2], where its rounding moves
+            // alpha by less than alpha's own last place (tau >= 1), and an error of the fast exponential only scales log alpha
+            const float sp = fmaxf(-z[i], 0.f) + logf(1.f + __expf(-fabsf(z[i])));
+            alpha[(size_t)(tb + i) * C + c] = expf(-sp * inv_tau);
+        }
 }
 
 // Row groups per column pair: the smallest power of two with DS * kRows >= rows.
@@ -623,9 +636,10 @@ XB_EXPORT int xb_linear_scan(float* o, const float* proj, long long ldp, const f
 XB_EXPORT int xb_low_rank_decay(float* alpha, const float* low, long long ldl, const float* w, const float* bias, int tokens,
                                 int C, int R, float tau, cudaStream_t stream) {
     if (tokens <= 0 || C <= 0) return 0;
-    if (R < 1 || !(tau > 0.f) || (C + 127) / 128 > 65535) return (int)cudaErrorInvalidValue;
-    const dim3 grid((tokens + kDecayTokens - 1) / kDecayTokens, (C + 127) / 128);
-    low_rank_decay_kernel<<<grid, 128, 0, stream>>>(alpha, low, ldl, w, bias, tokens, C, R, 1.f / tau);
+    const int cols = (C + kDecayChannels - 1) / kDecayChannels;
+    if (R < 1 || !(tau > 0.f) || cols > 65535) return (int)cudaErrorInvalidValue;
+    const dim3 grid((tokens + kDecayTokens - 1) / kDecayTokens, cols);
+    low_rank_decay_kernel<<<grid, kDecayChannels, 0, stream>>>(alpha, low, ldl, w, bias, tokens, C, R, 1.f / tau);
     return xb_launch_status();
 }
 

@@ -111,8 +111,20 @@ __global__ void __launch_bounds__(kThreads) stream_conv_kernel(TO* __restrict__ 
 #pragma unroll
         for (int v = 0; v < V; ++v) {
             bwv[v] = a.bw != nullptr ? (a.boffset + a.bw[c + v]) * a.bscale : a.bscale;
+        }
+        if (V == 4 && K % 4 == 0) {
 #pragma unroll
-            for (int j = 0; j < K; ++j) tap[j][v] = a.taps[(size_t)(c + v) * K + j];
+            for (int i = 0; i < K; ++i) {       // V * K neighbouring floats, four at a time
+                const float4 q = *reinterpret_cast<const float4*>(a.taps + (size_t)c * K + 4 * i);
+                const float e[4] = {q.x, q.y, q.z, q.w};
+#pragma unroll
+                for (int u = 0; u < 4; ++u) tap[(4 * i + u) % K][(4 * i + u) / K % V] = e[u];
+            }
+        } else {
+#pragma unroll
+            for (int v = 0; v < V; ++v)
+#pragma unroll
+                for (int j = 0; j < K; ++j) tap[j][v] = a.taps[(size_t)(c + v) * K + j];
         }
         // a row's sum at this thread's channels, from its parts
         auto sum_of = [&](int t, const float (&xv)[V], const float (&bv)[V], float (&s)[V]) {
@@ -264,17 +276,19 @@ XB_EXPORT int xb_stream_conv(int out_dtype, void* out, float* s_out, const float
     a.tokens = tokens; a.C = C; a.single = single;
     a.beps = beps; a.boffset = boffset; a.bscale = bscale;
     const size_t osz = out_dtype == XB_F32 ? 16 : 8;
-    const bool vec = C % 4 == 0 && !(((uintptr_t)x | (uintptr_t)branch | (uintptr_t)s_out | (uintptr_t)state) & 15) &&
+    const bool vec = C % 4 == 0 && !(((uintptr_t)x | (uintptr_t)branch | (uintptr_t)s_out | (uintptr_t)state | (uintptr_t)taps) & 15) &&
                      ((uintptr_t)out & (osz - 1)) == 0;
     // long runs pay for the rows before them only once, short ones fill the machine
     int run = kMaxRun;
     while (run > 1 && (tokens + run - 1) / run < 2 * 148) run /= 2;
     a.run = run;
     const int V = vec ? 4 : 1;
-    // with a norm every block of a row would reduce it again: one block takes all channels then
-    int cols = bw != nullptr ? 1 : (C + kThreads * V - 1) / (kThreads * V);
+    // with a norm every block of a row reduces it again: one block takes all channels then, but for steps of few tokens
+    const int runs = (tokens + run - 1) / run;
+    int cols = (C + kThreads * V - 1) / (kThreads * V);
+    if (bw != nullptr && runs >= 148) cols = 1;
     if (cols > 65535) cols = 65535;
-    const dim3 grid((tokens + run - 1) / run, cols);
+    const dim3 grid(runs, cols);
     typedef __nv_bfloat16 bf;
     if (out_dtype == XB_F32)
         return vec ? launch_taps<float, 4>((float*)out, a, K, grid, stream) : launch_taps<float, 1>((float*)out, a, K, grid, stream);
