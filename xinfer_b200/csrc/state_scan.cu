@@ -517,9 +517,7 @@ __global__ void __launch_bounds__(kDecayChannels) low_rank_decay_kernel(float* _
 #pragma unroll
     for (int i = 0; i < kDecayTokens; ++i)
         if (i < nt) {
-            // softplus(-z) without a branch.  What enters the sum's logarithm lies in (1, 2], where its rounding moves
-            // alpha by less than alpha's own last place (tau >= 1), and an error of the fast exponential only scales log alpha
-            const float sp = fmaxf(-z[i], 0.f) + logf(1.f + __expf(-fabsf(z[i])));
+            const float sp = fmaxf(-z[i], 0.f) + log1pf(expf(-fabsf(z[i])));      // softplus(-z), for any z without a branch
             alpha[(size_t)(tb + i) * C + c] = expf(-sp * inv_tau);
         }
 }
