@@ -7,12 +7,12 @@ import numpy as np
 from xinfer_b200.native import host_lib
 
 
-def work_list(counts, starts, dec_max, window, heads, kv_heads, max_ctas):
+def work_list(counts, starts, dec_max, window, 0, heads, kv_heads, max_ctas):
     counts, starts = np.asarray(counts, dtype=np.int32), np.asarray(starts, dtype=np.int32)
     cap = max_ctas + 1 + 4 * int(((counts + 127) // 128).sum()) * heads + 8
     out = np.full(cap, -9, dtype=np.int32)
     ctas = ctypes.c_int(0)
-    used = host_lib().xb_attn_prefill_work(len(counts), counts.ctypes.data, starts.ctypes.data, dec_max, window, heads, kv_heads,
+    used = host_lib().xb_attn_prefill_work(len(counts), counts.ctypes.data, starts.ctypes.data, dec_max, window, 0, heads, kv_heads,
                                            max_ctas, out.ctypes.data, cap, ctypes.byref(ctas))
     c = ctas.value
     offs = out[: c + 1]
@@ -67,5 +67,5 @@ def test_nothing_to_do_and_too_small_a_buffer():
     counts, starts = np.asarray([1000], dtype=np.int32), np.asarray([0], dtype=np.int32)
     out = np.zeros(10, dtype=np.int32)
     ctas = ctypes.c_int(0)
-    assert host_lib().xb_attn_prefill_work(1, counts.ctypes.data, starts.ctypes.data, 4, 0, 8, 2, 148, out.ctypes.data, 10,
+    assert host_lib().xb_attn_prefill_work(1, counts.ctypes.data, starts.ctypes.data, 4, 0, 0, 8, 2, 148, out.ctypes.data, 10,
                                            ctypes.byref(ctas)) == -1

@@ -18,11 +18,12 @@ from ..native import host_lib
 
 @dataclass(frozen=True)
 class CacheGroup:
-    """Layers whose caches grow alike: same page size, same retention (all keys or a window)."""
+    """Layers whose caches grow alike: same page size, same retention (all keys, or a window and perhaps the first positions)."""
 
     page_size: int
     num_pages: int
     window: Optional[int] = None  # None: keep every key
+    keep_first: int = 0           # beside a window: a sequence's first positions are kept too
 
 
 class CacheError(RuntimeError):
@@ -41,7 +42,7 @@ class CacheManager:
         self._lib = lib
         self._h = lib.xb_cm_create(
             n, arr(*[g.page_size for g in self.groups]), arr(*[g.num_pages for g in self.groups]),
-            arr(*[(g.window or 0) for g in self.groups]), self.max_requests)
+            arr(*[(g.window or 0) for g in self.groups]), arr(*[int(g.keep_first) for g in self.groups]), self.max_requests)
         if not self._h:
             raise CacheError(f"invalid cache groups {self.groups} / max_requests {max_requests}")
 

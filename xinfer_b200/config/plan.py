@@ -155,6 +155,17 @@ class AttentionSpec(PartSpec):
     # a query sees the earlier keys of its own chunk of this many positions (chunks counted from position 0 of the
     # sequence) instead of a window
     chunk: Optional[int] = None
+    # beside a window: the sequence's first ``keep_first`` positions stay visible (and cached) for ever
+    keep_first: int = 0
+    # the name of a learned score per head: one more entry of every softmax of the head, neither scaled nor masked, that
+    # carries no value
+    sink_name: Optional[str] = None
+    # taps of a causal convolution over time on every channel of the q, k and v projections, directly behind them
+    # (without a bias or an activation; filters: the matrix's name with ``conv_suffix``, ``[channels, taps]``)
+    conv: Optional[int] = None
+    conv_suffix: str = ".conv"
+    # values are divided by their root mean square per head before they are cached (this eps under the root, no weight)
+    value_norm_eps: Optional[float] = None
 
     @property
     def value_dim(self) -> int:
@@ -278,6 +289,26 @@ class GatedLinearAttentionSpec(PartSpec):
 
 
 @dataclass(frozen=True)
+class MatrixMemorySpec(PartSpec):
+    """A matrix memory with exponential gates in the form of xLSTM's mLSTM: q and k of ``heads x head_dim`` (q times
+    head_dim^-1/2), v of ``heads x v_head_dim``; per head a log input gate i = cap tanh((W_i h + b_i) / cap) and a log
+    forget gate f = logsigmoid(cap tanh((W_f h + b_f) / cap)), cap = ``gate_cap``; with a running maximum m that starts
+    at zero, m' = max(f + m, i), S <- e^(f + m - m') S + e^(i - m') k v^T, n likewise with k alone, and
+    o = S^T q / (max(|n . q|, e^(-m')) + ``divisor_eps``), read after the token's own write; o is RMS-normed per head
+    (``eps``) with a weight over all heads' channels, times sigmoid(W_g h), then projected out.  ``names``: q, k, v,
+    W_g, output, norm, W_i, b_i, W_f, b_f after the prefix."""
+
+    hidden: int = 0
+    heads: int = 0
+    head_dim: int = 0
+    v_head_dim: int = 0
+    gate_cap: float = 1.0
+    eps: float = 1e-6
+    divisor_eps: float = 1e-6
+    names: Tuple[str, ...] = ("q", "k", "v", "g", "o", "norm", "i", "i.b", "f", "f.b")
+
+
+@dataclass(frozen=True)
 class InputConvSpec(PartSpec):
     """A mixer whose input is first replaced by ``h + conv(h)``, a causal convolution of ``taps`` taps per channel
     (no bias, no activation) whose last ``taps - 1`` inputs are carried per request.  ``name``: the filter's tensor
@@ -380,6 +411,17 @@ class ExpertTableSpec(PartSpec):
 
 
 @dataclass(frozen=True)
+class StreamMixSpec:
+    """How half a layer reads and writes ``count`` residual streams X[0..count-1] (hyper-connections) with learned
+    numbers of its own: it reads ``u = sum_s r[s] X[s]`` and writes, all streams at once from the old ones,
+    ``X[t] <- sum_s M[s, t] X[s] + w[t] y``.  ``names``: r ``[count]``, M ``[count, count]`` (from, to) and w ``[count]``
+    after the block's prefix."""
+
+    count: int
+    names: Tuple[str, str, str]
+
+
+@dataclass(frozen=True)
 class BlockOp:
     """One operation of a block's program.  A program works on named activations of shape
     ``[tokens, hidden]``; ``"x"`` is the residual stream that enters and leaves the block, every
@@ -389,6 +431,9 @@ class BlockOp:
     * ``op="mixer"`` / ``op="feed_forward"``: ``dst = part(src)`` with the part ``spec``;
     * ``op="add"``: ``dst = dst + scale * gain * src`` (no spec); ``gain`` names a learned vector over the
       channels (its tensor name after the block's prefix; None: ones).
+
+    ``mix``: the residual stream is several streams; a norm of ``"x"`` reads their weighted sum and an addition into
+    ``"x"`` mixes them and adds to each (``StreamMixSpec``).
 
     ``name`` is the tensor-name piece between the block's prefix and the part's own tensor names;
     two operations with the same ``op`` and ``name`` are the same part (one set of weights).
@@ -404,6 +449,7 @@ class BlockOp:
     name: str = ""
     scale: float = 1.0
     gain: Optional[str] = None
+    mix: Optional[StreamMixSpec] = None
 
 
 BLOCK_OPS = ("norm", "mixer", "feed_forward", "add")
@@ -432,12 +478,18 @@ class BlockSpec:
         ops = self.ops_of("feed_forward")
         return ops[0].spec if ops else None
 
+    @property
+    def streams(self) -> Optional[int]:
+        """The number of residual streams, None for the one plain stream."""
+        return next((o.mix.count for o in self.program if o.mix is not None), None)
+
     def norms(self) -> Tuple[PartSpec, ...]:
         return tuple(o.spec for o in self.ops_of("norm"))
 
     def validate(self) -> None:
         defined = {"x"}
         mixers = set()
+        counts = set()        # numbers of residual streams the operations on them name (None: the one plain stream)
         for i, o in enumerate(self.program):
             where = f"block '{self.prefix}' operation {i} ({o.op})"
             if o.op not in BLOCK_OPS:
@@ -461,6 +513,17 @@ class BlockSpec:
                 defined.add(o.dst)
             if o.op == "mixer":
                 mixers.add(o.name)
+            touches_x = (o.src == "x" and o.op != "add") or (o.dst == "x" and o.op == "add")
+            if o.mix is not None:
+                if not touches_x or o.op not in ("norm", "add") or (o.op == "norm" and o.dst == "x"):
+                    raise ValueError(f"{where}: only a norm of the residual stream and an addition into it deal with "
+                                     f"several streams")
+                if o.mix.count < 1 or o.scale != 1.0 or o.gain is not None:
+                    raise ValueError(f"{where}: streams are mixed without a scale or a gain, and there is at least one")
+            if touches_x or "x" in (o.src, o.dst):
+                counts.add(o.mix.count if o.mix is not None else None)
+        if len(counts) > 1:
+            raise ValueError(f"block '{self.prefix}': its operations disagree about the number of residual streams")
         if len(mixers) > 1:
             raise ValueError(f"block '{self.prefix}' holds {len(mixers)} mixers; a block holds at most one "
                              f"(write the layer as several blocks)")
@@ -529,6 +592,9 @@ class ModelPlan:
     # learned vector per position (the tensor's name; it has max_positions rows)
     pair_embedding: Optional["PairEmbeddingSpec"] = None
     position_table: Optional[str] = None
+    # how many residual streams there are, all equal to the embedding's output at first and summed before the final
+    # norm (None: one plain stream)
+    streams: Optional[int] = None
     # standard deviations used by the random-weights mode
     init_std: float = 0.02
     norm_init_std: float = 0.1
@@ -544,6 +610,10 @@ class ModelPlan:
             raise ValueError("a pair embedding or a position table is summed into a float32 residual stream")
         if self.logit_softcap is not None and not (self.logit_softcap > 0):
             raise ValueError(f"logit_softcap must be positive, got {self.logit_softcap}")
+        if any(b.streams != self.streams for b in self.blocks):
+            raise ValueError("the model and its blocks disagree about the number of residual streams")
+        if self.streams is not None and (self.residual_dtype != "float32" or any(r.add_input for r in self.runs)):
+            raise ValueError("several residual streams are float32, and no run adds the embedding to them again")
         for pos, run in enumerate(self.runs):
             if not (0 <= run.block < len(self.blocks)):
                 raise ValueError(f"run {pos} names block {run.block}, but there are {len(self.blocks)}")

@@ -86,12 +86,14 @@ def _register_builtin() -> None:
     from .gulipel import GulipelConfig
     from .mikutar import MikutarConfig
     from .napuzen import NapuzenConfig
+    from .dalalix import DalalixConfig
     register_architecture(Qwen3Config.ARCHITECTURE, Qwen3Config.from_dict, lambda c: c.plan())
     register_architecture(TidaraxConfig.ARCHITECTURE, TidaraxConfig.from_dict, lambda c: c.plan())
     register_architecture(DufitarConfig.ARCHITECTURE, DufitarConfig.from_dict, lambda c: c.plan())
     register_architecture(GulipelConfig.ARCHITECTURE, GulipelConfig.from_dict, lambda c: c.plan())
     register_architecture(MikutarConfig.ARCHITECTURE, MikutarConfig.from_dict, lambda c: c.plan())
     register_architecture(NapuzenConfig.ARCHITECTURE, NapuzenConfig.from_dict, lambda c: c.plan())
+    register_architecture(DalalixConfig.ARCHITECTURE, DalalixConfig.from_dict, lambda c: c.plan())
 
 
 _register_builtin()

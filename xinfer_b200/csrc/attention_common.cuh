@@ -26,6 +26,15 @@ __host__ __device__ __forceinline__ int first_visible(int pos, int mask) {
     return 0;
 }
 
+// Beside a sliding window a query may go on seeing the first `keep` positions of its sequence.  The keys it sees are
+// then walked over in two pieces: the `kept_tiles` tiles of `tile` keys from position 0 that hold them and lie before the
+// tile of the window's first key `lo`, then the window's own.  tile_at: the n-th tile of that walk.
+__host__ __device__ __forceinline__ int kept_tiles(int keep, int lo, int tile) {
+    const int a = (keep + tile - 1) / tile, b = lo / tile;
+    return keep > 0 ? (a < b ? a : b) : 0;
+}
+__host__ __device__ __forceinline__ int tile_at(int n, int kept, int lo, int tile) { return n < kept ? n : lo / tile + n - kept; }
+
 // Scores that are changed before the softmax: s <- cap * tanh(s / cap) (cap > 0), then s <- s - slope * dist for a
 // key dist positions back.  With e = exp(2 s / cap), cap * tanh(s / cap) = cap - 2 cap / (e + 1): one exponential, one
 // reciprocal and one multiply-add that also takes whatever is added to the score (absolute error about 1e-7 of the

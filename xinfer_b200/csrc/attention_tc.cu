@@ -59,13 +59,13 @@ constexpr int PREFILL_ITEM_INTS = 4;   // portion, query tile, first query head,
 struct PrefillItem {
     int g, h0, nhd;               // key/value head, first query head, heads (2, or 1)
     int rows, t0, p0;             // queries, their first row in q / out, the first one's position
-    int first_key, last_key, kt_first, iters;
+    int first_key, last_key, kept, iters;   // kept: key tiles of the sequence's first positions, ahead of the window's
     const int* table;
 };
 
 __device__ __forceinline__ PrefillItem prefill_item(const int* __restrict__ item, const int* __restrict__ q_start,
                                                     const int* __restrict__ start_pos, const int* __restrict__ block_table,
-                                                    int table_stride, int nh, int nkv, int window) {
+                                                    int table_stride, int nh, int nkv, int window, int keep) {
     PrefillItem w;
     const int b = item[0], tile = item[1];
     w.h0 = item[2];
@@ -81,8 +81,8 @@ __device__ __forceinline__ PrefillItem prefill_item(const int* __restrict__ item
     w.last_key = w.p0 + w.rows - 1;
     w.first_key = first_visible(w.p0, window);
     w.table = block_table + (size_t)b * table_stride;
-    w.kt_first = w.first_key / KT;
-    w.iters = w.last_key / KT - w.kt_first + 1;
+    w.kept = kept_tiles(keep, w.first_key, KT);
+    w.iters = w.kept + w.last_key / KT - w.first_key / KT + 1;
     return w;
 }
 
@@ -93,8 +93,9 @@ __global__ void __launch_bounds__(PREFILL_THREADS)
 attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                        const __grid_constant__ CUtensorMap map_v, const __grid_constant__ CUtensorMap map_o,
                        __nv_bfloat16* __restrict__ out, const int* __restrict__ q_start, const int* __restrict__ start_pos,
-                       const int* __restrict__ block_table, int table_stride, int nh, int nkv, int d,
-                       int ps, int ps_shift, int num_pages, int window, float scale_log2_in, float softcap, float slope_exp,
+                       const int* __restrict__ block_table, int table_stride, int nh, int nkv, int dv, long long ldo,
+                       int ps, int ps_shift, int num_pages, int window, int keep, float scale_log2_in, float softcap,
+                       float slope_exp, const float* __restrict__ sink, float out_scale,
                        const int* __restrict__ work, int* err) {
     // changed scores (a cap, a bias on the distance): the scores are brought to their final values first and the
     // softmax then only changes the base of the exponential
@@ -155,7 +156,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
 
     const int box_rows = ps < KT ? ps : KT;
     auto item_at = [&](int k) {
-        return prefill_item(items + (size_t)k * PREFILL_ITEM_INTS, q_start, start_pos, block_table, table_stride, nh, nkv, window);
+        return prefill_item(items + (size_t)k * PREFILL_ITEM_INTS, q_start, start_pos, block_table, table_stride, nh, nkv, window, keep);
     };
     if (warp == 8 || warp == 10) {
         // ---- producers of key pages (warp 8) and value pages (warp 10), item after item ----------------------
@@ -171,8 +172,8 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
             const int boxes = (KT / box_rows) * HALVES;     // at most 16: one lane each
             const int bi = lane / HALVES, hf = lane % HALVES;
             auto page_of = [&](int it) -> int {             // the page of this lane's box in tile `it`, -1: nothing to load
-                const int j = (w.kt_first + it) * KT + bi * box_rows;
-                if (it >= w.iters || lane >= boxes || j > w.last_key || j + box_rows - 1 < w.first_key) return -1;
+                const int j = tile_at(it, w.kept, w.first_key, KT) * KT + bi * box_rows;
+                if (it >= w.iters || lane >= boxes || j > w.last_key || (j + box_rows - 1 < w.first_key && j >= keep)) return -1;
                 const int page = w.table[j >> ps_shift];
                 if (page < 0 || page >= num_pages) {
                     atomicOr(err, XB_ERR_BAD_PAGE);
@@ -193,7 +194,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
                 if (lane == 0) mbar_expect_tx(full0 + 8 * s, nb * box_rows * 128);
                 __syncwarp();
                 if (page >= 0) {
-                    const int j = (w.kt_first + it) * KT + bi * box_rows;
+                    const int j = tile_at(it, w.kept, w.first_key, KT) * KT + bi * box_rows;
                     const uint32_t dst = kv_sm + s * STAGE_BYTES + (is_v ? KV_BYTES : 0u) + hf * KV_HALF + bi * box_rows * 128;
                     tma_load_2d(dst, map, hf * 64, (page * nkv + w.g) * ps + (j & (ps - 1)), full0 + 8 * s);
                 }
@@ -345,14 +346,14 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
                 T += w.iters;
                 continue;
             }
-            const int iters = w.iters, kt_first = w.kt_first, first_key = w.first_key, last_key = w.last_key, p0 = w.p0;
+            const int iters = w.iters, kept = w.kept, first_key = w.first_key, last_key = w.last_key, p0 = w.p0;
             const int rows = w.rows, t0 = w.t0, h0 = w.h0;
             const int my_pos = p0 + r;
             const int my_lo = first_visible(my_pos, window), edge_lo = first_visible(p0 + QT - 1, window);
             const float slope = head_slope(slope_exp, h0 + hd, nh);
             float m_ref = -INFINITY, l = 0.f;
             for (int it = 0; it < iters; ++it) {
-                const int th = Th + it, sb = th & 1, gt = T + it, st = gt % NS, key0 = (kt_first + it) * KT;
+                const int th = Th + it, sb = th & 1, gt = T + it, st = gt % NS, key0 = tile_at(it, kept, first_key, KT) * KT;
                 // every wait's verdict is made warp-wide: tcgen05.ld / .st below need the whole warp
                 if (!__all_sync(0xffffffffu, mbar_wait(my_s_ready + 8 * sb, (th >> 1) & 1, err))) {
                     alive = false;
@@ -382,13 +383,13 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
                         for (int i = 0; i < 64; ++i) sc[i] = fmaf(slope, (float)i, fmaf(sc[i], scale_nat, base));
                     }
                 }
-                const bool edge = key0 + KT - 1 > p0 || key0 + KT - 1 > last_key || key0 < first_key || key0 < edge_lo;
+                const bool edge = key0 + KT - 1 > p0 || key0 + KT - 1 > last_key || (key0 < edge_lo && key0 + KT > keep);
                 float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
                 if (edge) {
     #pragma unroll
                     for (int i = 0; i < 64; ++i) {
                         const int j = key0 + i;
-                        const bool ok = j <= my_pos && j <= last_key && j >= my_lo;
+                        const bool ok = j <= my_pos && j <= last_key && (j >= my_lo || j < keep);
                         sc[i] = ok ? sc[i] : -INFINITY;
                     }
                 }
@@ -438,11 +439,11 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
                 tmem_st32_u(tmem_s + sb * 64 + lane_addr, pk);
                 // value rows outside the visible keys become zeros (only tiles at the ends of the range): the first
                 // head's threads do it; the second head's P V is issued after the first's, so it sees them too
-                if (hd == 0 && (key0 < first_key || key0 + KT - 1 > last_key)) {
+                if (hd == 0 && ((key0 < first_key && key0 + KT > keep) || key0 + KT - 1 > last_key)) {
                     if (r < KT) {
                         mbar_wait(v_full0 + 8 * st, (gt / NS) & 1, err);   // orders these writes after the TMA's
                         const int j = key0 + r;
-                        if (j < first_key || j > last_key) {
+                        if ((j < first_key && j >= keep) || j > last_key) {
     #pragma unroll
                             for (int hf = 0; hf < HALVES; ++hf) {
                                 uint4* vr = reinterpret_cast<uint4*>(smem_raw + Q_BYTES + st * STAGE_BYTES + KV_BYTES + hf * KV_HALF + r * 128);
@@ -482,11 +483,13 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
             if (alive) alive = mbar_wait(bar_o, (uint32_t)I & 1u, err);
             alive = __all_sync(0xffffffffu, alive);
             asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+            // a sink: one more entry of the denominator, at the score it is given (a row that sees no key: nothing)
+            if (sink != nullptr) l += exp2f(fmaf(sink[h0 + hd], 1.4426950408889634f, -m_ref));
+            const float inv = l > 0.f ? out_scale / l : 0.f;
             if (alive && rows == QT) {
                 // a full tile: a warp writes its 32 rows of a 64-column half, swizzled, into its staging space and
                 // one thread stores them with a TMA copy: whole lines reach the memory instead of 16 bytes per row
                 // and instruction.  Meanwhile the issuers are at work on the next item.
-                const float inv = l > 0.f ? 1.f / l : 0.f;
                 const int rr = lane;   // row within the warp's 32
                 if (lane == 0) tma_store_wait_read();   // the stores of this warp's item before have read the staging space
                 __syncwarp();
@@ -510,13 +513,12 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
                 if (lane == 0) {
 #pragma unroll
                     for (int hf = 0; hf < HALVES; ++hf)
-                        if (hf * 64 < d) tma_store_3d(&map_o, stage_sm + hf * 4096, hf * 64, h0 + hd, t0 + (warp & 3) * 32);
+                        if (hf * 64 < dv) tma_store_3d(&map_o, stage_sm + hf * 4096, hf * 64, h0 + hd, t0 + (warp & 3) * 32);
                     tma_store_commit();
                 }
             } else if (alive) {
-                const float inv = l > 0.f ? 1.f / l : 0.f;
                 const bool valid = r < rows;
-                __nv_bfloat16* dst = out + ((size_t)(t0 + r) * nh + h0 + hd) * d;
+                __nv_bfloat16* dst = out + (size_t)(t0 + r) * ldo + (size_t)(h0 + hd) * dv;
 #pragma unroll
                 for (int c0 = 0; c0 < DP; c0 += 32) {
                     float o[32];
@@ -525,7 +527,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
 #pragma unroll
                         for (int c8 = 0; c8 < 4; ++c8) {
                             const int c = c0 + c8 * 8;
-                            if (c < d) {
+                            if (c < dv) {
                                 uint4 pk;
                                 pk.x = pack_bf16(o[c8 * 8] * inv, o[c8 * 8 + 1] * inv);
                                 pk.y = pack_bf16(o[c8 * 8 + 2] * inv, o[c8 * 8 + 3] * inv);
@@ -560,7 +562,7 @@ constexpr int DEC_ROWS = 16;    // query heads of one key/value head a CTA can h
 // latency at full rate, so twice as many where a tile is half as large
 __host__ __device__ constexpr int dec_stages(int dp) { return dp <= 64 ? 6 : 3; }
 constexpr int PLAN_HEADER = 4;  // int32 before the first piece of a plan: [0] = number of pieces
-constexpr int PLAN_ENTRY = 8;   // int32 per piece: token row, request, position, first key, first tile, tiles,
+constexpr int PLAN_ENTRY = 8;   // int32 per piece: token row, request, position, the window's first key, first of its tiles (in the walk), tiles,
                                 // pieces of the token << 16 | index of this one, rank of the token among the small ones
 constexpr int PLAN_THREADS = 512;
 constexpr int PLAN_SORT_MAX = 1024;   // up to this many pieces are put in order of their length, longest first
@@ -574,7 +576,7 @@ constexpr int PLAN_TOKENS_MAX = 16 * PLAN_THREADS;
 __global__ void __launch_bounds__(PLAN_THREADS)
 attn_decode_plan_kernel(int* __restrict__ plan, int capacity, const int* __restrict__ positions,
                         const int* __restrict__ req_of_token, const int* __restrict__ q_start, int num_entries, int window,
-                        int dec_max, int direct, int num_small, int min_tiles, int target_ctas, int nkv, int* err) {
+                        int keep, int dec_max, int direct, int num_small, int min_tiles, int target_ctas, int nkv, int* err) {
     __shared__ int warp_sums[PLAN_THREADS / 32];
     __shared__ int piece_tiles[PLAN_SORT_MAX];
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
@@ -609,7 +611,7 @@ attn_decode_plan_kernel(int* __restrict__ plan, int capacity, const int* __restr
             if (t >= 0 && req_of_token[t] >= 0) {
                 const int pos = positions[t];
                 const int lo = first_visible(pos, window);
-                tiles[i] = pos / KT - lo / KT + 1;
+                tiles[i] = kept_tiles(keep, lo, KT) + pos / KT - lo / KT + 1;
                 tok[i] = t;
             }
         }
@@ -664,7 +666,7 @@ attn_decode_plan_kernel(int* __restrict__ plan, int capacity, const int* __restr
             e[1] = req_of_token[t];
             e[2] = pos;
             e[3] = lo;
-            e[4] = lo / KT + i0;
+            e[4] = i0;
             e[5] = i0 < n ? min(sz, n - i0) : 0;   // an empty piece (rounding): its CTA leaves
             e[6] = (ns << 16) | j;
             e[7] = z;
@@ -689,8 +691,9 @@ __global__ void __launch_bounds__(128)
 attn_decode_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                       const __grid_constant__ CUtensorMap map_v, __nv_bfloat16* __restrict__ out,
                       float* __restrict__ part_o, float* __restrict__ part_ml, const int* __restrict__ plan,
-                      const int* __restrict__ block_table, int table_stride, int nh, int nkv, int d, int ps,
-                      int ps_shift, int num_pages, float scale_log2_in, float softcap, float slope_exp, int dec_max,
+                      const int* __restrict__ block_table, int table_stride, int nh, int nkv, int dv, long long ldo, int ps,
+                      int ps_shift, int num_pages, int keep, float scale_log2_in, float softcap, float slope_exp,
+                      const float* __restrict__ sink, float out_scale, int dec_max,
                       int splits_max, int page_cap, int* __restrict__ tickets, int* err) {
     constexpr int HALVES = DP / 64, DEC_STAGES = dec_stages(DP);
     // changed scores (a cap, a bias on the distance): brought to their final values before the softmax, which then
@@ -724,19 +727,20 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
     if ((int)blockIdx.y >= plan[0]) return;
     const int4 e0 = __ldg(reinterpret_cast<const int4*>(plan + PLAN_HEADER) + 2 * blockIdx.y);
     const int4 e1 = __ldg(reinterpret_cast<const int4*>(plan + PLAN_HEADER) + 2 * blockIdx.y + 1);
-    const int t = e0.x, b = e0.y, pos = e0.z, lo = e0.w, kt_first = e1.x, z = e1.w;
+    const int t = e0.x, b = e0.y, pos = e0.z, lo = e0.w, walk0 = e1.x, z = e1.w;
     const int ns = e1.z >> 16, slot = e1.z & 0xFFFF;
     if (e1.y <= 0) return;
-    const int kt_last = kt_first + e1.y - 1;
-    const int k_begin = max(lo, kt_first * KT), k_end = min(pos, kt_last * KT + KT - 1);
+    const int iters = e1.y, kept = kept_tiles(keep, lo, KT);
+    auto tile_of = [&](int it) { return tile_at(walk0 + it, kept, lo, KT); };   // the piece's tiles, in order
     const int fresh = pos - dec_max + 1;   // keys before this were written by earlier steps, not by the kernel before this one
     const int* table = block_table + (size_t)b * table_stride;
     const int h0 = g * G;
-    const int iters = kt_last - kt_first + 1;
-    const int box_rows = ps < KT ? ps : KT;
-    const int page_first = (kt_first * KT) >> ps_shift;
-    const int staged = min((k_end >> ps_shift) - page_first + 1, page_cap);
-    for (int i = threadIdx.x; i < staged; i += 128) s_pages[i] = table[page_first + i];
+    const int box_rows = ps < KT ? ps : KT, box_shift = ps < KT ? 6 - ps_shift : 0;   // KT is 1 << box_shift boxes
+    const int staged = min(iters << box_shift, page_cap);      // the page of every box of the piece
+    for (int i = threadIdx.x; i < staged; i += 128) {
+        const int j = tile_of(i >> box_shift) * KT + (i & ((1 << box_shift) - 1)) * box_rows;
+        s_pages[i] = j <= pos ? table[j >> ps_shift] : -1;
+    }
 
     if (threadIdx.x == 0) {
         if (base & 1023u) atomicOr(err, XB_ERR_WAIT);  // the swizzle needs a 1024-byte aligned window
@@ -776,12 +780,12 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
         const int boxes = (KT / box_rows) * HALVES;
         const int bi = lane / HALVES, hf = lane % HALVES;
         auto issue_tile = [&](int it) {
-            const int s = it % DEC_STAGES, kt = kt_first + it;
+            const int s = it % DEC_STAGES, kt = tile_of(it);
             const uint32_t dst = kv_sm + s * STAGE_BYTES + (is_v ? KV_BYTES : 0u) + hf * KV_HALF + bi * box_rows * 128;
             const int j = kt * KT + bi * box_rows;
             int page = -1;
-            if (lane < boxes && j <= k_end && j + box_rows - 1 >= k_begin) {
-                const int idx = (j >> ps_shift) - page_first;
+            if (lane < boxes && j <= pos && (j + box_rows - 1 >= lo || j < keep)) {
+                const int idx = (it << box_shift) + bi;
                 page = idx < staged ? s_pages[idx] : table[j >> ps_shift];
                 if (page < 0 || page >= num_pages) {
                     atomicOr(err, XB_ERR_BAD_PAGE);
@@ -795,7 +799,7 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
         };
         // tiles that hold only keys of earlier steps do not depend on the kernel before this one
         int pre = 0;
-        while (pre < iters && pre < DEC_STAGES && (kt_first + pre) * KT + KT - 1 < fresh) issue_tile(pre++);
+        while (pre < iters && pre < DEC_STAGES && tile_of(pre) * KT + KT - 1 < fresh) issue_tile(pre++);
         pdl_wait();
         if (!is_v && lane == 0) {
             mbar_expect_tx(q_full, HALVES * G * 128);
@@ -858,7 +862,7 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
         float m_ref[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
         bool alive = true;
         for (int it = 0; it < iters; ++it) {
-            const int s = it & 1, key0 = (kt_first + it) * KT;
+            const int s = it & 1, key0 = tile_of(it) * KT;
             if (!__all_sync(0xffffffffu, mbar_wait(s_ready0 + 8 * s, (it >> 1) & 1, err))) {
                 alive = false;
                 break;
@@ -868,7 +872,7 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
             tmem_ld_16x256b_x8(tmem_s + s * 64, raw);
             asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
             mbar_arrive(s_free0 + 8 * s);   // S[s] is in registers
-            const bool edge = key0 < k_begin || key0 + KT - 1 > k_end;
+            const bool edge = (key0 < lo && key0 + KT > keep) || key0 + KT - 1 > pos;
             float corr[2] = {1.f, 1.f};
             int moved = 0;
             uint32_t pk[2][8];
@@ -890,7 +894,7 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
                         }
                         if (edge) {
                             const int j = key0 + 8 * k + 2 * quad + e;
-                            v = (j >= k_begin && j <= k_end) ? v : -INFINITY;
+                            v = ((j >= lo || j < keep) && j <= pos) ? v : -INFINITY;
                         }
                         sc[2 * k + e] = v;
                         mx2[e] = fmaxf(mx2[e], v);
@@ -939,7 +943,7 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
 #pragma unroll
                 for (int rr = 0; rr < 2; ++rr) {
                     const int row = lane + rr * 32, j = key0 + row;
-                    if (j < k_begin || j > k_end) {
+                    if ((j < lo && j >= keep) || j > pos) {
 #pragma unroll
                         for (int hf = 0; hf < HALVES; ++hf) {
                             uint4* vr = reinterpret_cast<uint4*>(v_ptr + hf * KV_HALF + row * 128);
@@ -982,9 +986,12 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
         const float ma = __shfl_sync(0xffffffffu, m_ref[0], (lane & 7) * 4), mb = __shfl_sync(0xffffffffu, m_ref[1], (lane & 7) * 4);
         if (alive) {
             const float l_row = lane < 8 ? la : lb, m_row = lane < 8 ? ma : mb;
-            const float inv = l_row > 0.f ? 1.f / l_row : 0.f;
             const bool valid = lane < G && ns <= splits_max;
             const int h = h0 + lane;
+            // a sink is one more entry of the denominator; it counts once, where a token's pieces come together
+            float l_all = l_row;
+            if (sink != nullptr && ns == 1 && lane < G) l_all += exp2f(fmaf(sink[h], 1.4426950408889634f, -m_row));
+            const float inv = l_all > 0.f ? (ns == 1 ? out_scale : 1.f) / l_all : 0.f;
             const size_t pslot = ((size_t)z * nh + h) * splits_max + slot;   // by the token's rank among the small ones
 #pragma unroll
             for (int c0 = 0; c0 < DP; c0 += 32) {
@@ -992,11 +999,11 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
                 tmem_ld32(tmem_o + c0, o);   // warp-wide, whatever `valid` is
                 if (!valid) continue;
                 if (ns == 1) {
-                    __nv_bfloat16* dst = out + ((size_t)t * nh + h) * d;
+                    __nv_bfloat16* dst = out + (size_t)t * ldo + (size_t)h * dv;
 #pragma unroll
                     for (int c8 = 0; c8 < 4; ++c8) {
                         const int c = c0 + c8 * 8;
-                        if (c < d) {
+                        if (c < dv) {
                             uint4 w;
                             w.x = pack_bf16(o[c8 * 8] * inv, o[c8 * 8 + 1] * inv);
                             w.y = pack_bf16(o[c8 * 8 + 2] * inv, o[c8 * 8 + 3] * inv);
@@ -1006,11 +1013,11 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
                         }
                     }
                 } else {
-                    float* dst = part_o + pslot * d;
+                    float* dst = part_o + pslot * dv;
 #pragma unroll
                     for (int c4 = 0; c4 < 8; ++c4) {
                         const int c = c0 + c4 * 4;
-                        if (c < d)
+                        if (c < dv)
                             *reinterpret_cast<float4*>(dst + c) = make_float4(o[c4 * 4] * inv, o[c4 * 4 + 1] * inv, o[c4 * 4 + 2] * inv, o[c4 * 4 + 3] * inv);
                     }
                 }
@@ -1062,7 +1069,7 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
                 float4 v[8];
 #pragma unroll
                 for (int i = 0; i < 8; ++i)
-                    v[i] = (i0 + i < ns && c4 < d) ? __ldcg(reinterpret_cast<const float4*>(part_o + (pbase + i0 + i) * d + c4))
+                    v[i] = (i0 + i < ns && c4 < dv) ? __ldcg(reinterpret_cast<const float4*>(part_o + (pbase + i0 + i) * dv + c4))
                                                    : make_float4(0.f, 0.f, 0.f, 0.f);
                 if (i0 == 0) {
                     M = warp_max(mi);
@@ -1077,9 +1084,10 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
                     }
                 }
             }
-            const float inv = W > 0.f ? 1.f / W : 0.f;
-            if (c4 < d) {
-                __nv_bfloat16* dst = out + ((size_t)t * nh + h) * d + c4;
+            if (sink != nullptr) W += exp2f(fmaf(sink[h], 1.4426950408889634f, -M));
+            const float inv = W > 0.f ? out_scale / W : 0.f;
+            if (c4 < dv) {
+                __nv_bfloat16* dst = out + (size_t)t * ldo + (size_t)h * dv + c4;
                 *reinterpret_cast<uint32_t*>(dst) = pack_bf16(acc.x * inv, acc.y * inv);
                 *reinterpret_cast<uint32_t*>(dst + 2) = pack_bf16(acc.z * inv, acc.w * inv);
             }
@@ -1091,17 +1099,18 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
         float wloc = 0.f;
         for (int i = lane; i < ns; i += 32)
             wloc += __ldcg(part_ml + (pbase + i) * 2 + 1) * exp2f(__ldcg(part_ml + (pbase + i) * 2) - M);
-        const float W = warp_sum(wloc);
-        const float inv = W > 0.f ? 1.f / W : 0.f;
-        for (int c4 = lane * 4; c4 < d; c4 += 128) {
+        float W = warp_sum(wloc);
+        if (sink != nullptr) W += exp2f(fmaf(sink[h], 1.4426950408889634f, -M));
+        const float inv = W > 0.f ? out_scale / W : 0.f;
+        for (int c4 = lane * 4; c4 < dv; c4 += 128) {
             float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll 8
             for (int i = 0; i < ns; ++i) {
                 const float w = __ldcg(part_ml + (pbase + i) * 2 + 1) * exp2f(__ldcg(part_ml + (pbase + i) * 2) - M);
-                const float4 v = __ldcg(reinterpret_cast<const float4*>(part_o + (pbase + i) * d + c4));
+                const float4 v = __ldcg(reinterpret_cast<const float4*>(part_o + (pbase + i) * dv + c4));
                 acc.x += v.x * w; acc.y += v.y * w; acc.z += v.z * w; acc.w += v.w * w;
             }
-            __nv_bfloat16* dst = out + ((size_t)t * nh + h) * d + c4;
+            __nv_bfloat16* dst = out + (size_t)t * ldo + (size_t)h * dv + c4;
             *reinterpret_cast<uint32_t*>(dst) = pack_bf16(acc.x * inv, acc.y * inv);
             *reinterpret_cast<uint32_t*>(dst + 2) = pack_bf16(acc.z * inv, acc.w * inv);
         }
@@ -1113,42 +1122,44 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
 bool map_rows(CUtensorMap* out, const void* ptr, long long rows, int d, int box_rows) {
     return tensor_map_2d(out, ptr, rows, d, box_rows);
 }
-// q [T, nh, d] through boxes [box_tokens x box_heads x 64 columns].
-bool map_q3(CUtensorMap* out, const void* ptr, long long T, int nh, int d, int box_heads, int box_tokens) {
-    const long long dims[3] = {d, nh, T}, strides[2] = {d, (long long)nh * d};
+// q [T, nh, d] (tokens ld elements apart) through boxes [box_tokens x box_heads x 64 columns].
+bool map_q3(CUtensorMap* out, const void* ptr, long long T, int nh, int d, long long ld, int box_heads, int box_tokens) {
+    const long long dims[3] = {d, nh, T}, strides[2] = {d, ld};
     const int box[3] = {64, box_heads, box_tokens};
     return tensor_map_bf16(out, ptr, 3, dims, strides, box);
 }
 
 template <int DP>
 int launch_prefill(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, const CUtensorMap& mo, void* out,
-                   const int* q_start, const int* start_pos, const int* table, int stride, int nh, int nkv, int d, int ps,
-                   int ps_shift, int num_pages, int window, float sl2, float softcap, float slope_exp, const int* work, int ctas,
-                   int* err, cudaStream_t stream) {
+                   const int* q_start, const int* start_pos, const int* table, int stride, int nh, int nkv, int dv,
+                   long long ldo, int ps, int ps_shift, int num_pages, int window, int keep, float sl2, float softcap,
+                   float slope_exp, const float* sink, float out_scale, const int* work, int ctas, int* err,
+                   cudaStream_t stream) {
     // Q of two heads, the key/value stages, the barriers' kilobyte, 4 KB of output staging per softmax warp and half
     constexpr size_t smem = 2 * (size_t)(DP / 64) * QT * 128 + PREFILL_STAGES * 2 * (size_t)(DP / 64) * KT * 128 + 1024 +
                             8 * (size_t)(DP / 64) * 4096;
     cudaFuncSetAttribute(attn_prefill_tc_kernel<DP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     cudaFuncSetAttribute(attn_prefill_tc_kernel<DP>, cudaFuncAttributePreferredSharedMemoryCarveout, 100);
     return xb_launch(attn_prefill_tc_kernel<DP>, dim3(ctas), dim3(PREFILL_THREADS), smem, stream, mq, mk, mv, mo,
-                     (__nv_bfloat16*)out, q_start, start_pos, table, stride, nh, nkv, d, ps, ps_shift, num_pages,
-                     window, sl2, softcap, slope_exp, work, err);
+                     (__nv_bfloat16*)out, q_start, start_pos, table, stride, nh, nkv, dv, ldo, ps, ps_shift, num_pages,
+                     window, keep, sl2, softcap, slope_exp, sink, out_scale, work, err);
 }
 
-constexpr int DEC_PAGE_CAP = 1024;   // block-table entries of a piece that are staged in shared memory
+constexpr int DEC_PAGE_CAP = 1024;   // page boxes of a piece whose pages are staged in shared memory
 
 template <int DP>
 int launch_decode(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, void* out, float* part_o,
-                  float* part_ml, const int* plan, int pieces, const int* table, int stride, int nh, int nkv, int d, int ps,
-                  int ps_shift, int num_pages, float sl2, float softcap, float slope_exp, int dec_max, int splits_max,
-                  int* tickets, int overlap, int* err, cudaStream_t stream) {
+                  float* part_ml, const int* plan, int pieces, const int* table, int stride, int nh, int nkv, int dv,
+                  long long ldo, int ps, int ps_shift, int num_pages, int keep, float sl2, float softcap, float slope_exp,
+                  const float* sink, float out_scale, int dec_max, int splits_max, int* tickets, int overlap, int* err,
+                  cudaStream_t stream) {
     constexpr size_t smem = (size_t)(DP / 64) * DEC_ROWS * 128 + 2 * DEC_ROWS * 128 + dec_stages(DP) * 2 * (size_t)(DP / 64) * KT * 128 +
                             32 * dec_stages(DP) + 96 + (size_t)DEC_PAGE_CAP * 4;
     cudaFuncSetAttribute(attn_decode_tc_kernel<DP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     cudaFuncSetAttribute(attn_decode_tc_kernel<DP>, cudaFuncAttributePreferredSharedMemoryCarveout, 100);
     return xb_launch_opt(overlap != 0, attn_decode_tc_kernel<DP>, dim3(nkv, pieces), dim3(128), smem, stream, mq, mk, mv,
-                         (__nv_bfloat16*)out, part_o, part_ml, plan, table, stride, nh, nkv, d, ps, ps_shift, num_pages, sl2,
-                         softcap, slope_exp, dec_max, splits_max, DEC_PAGE_CAP, tickets, err);
+                         (__nv_bfloat16*)out, part_o, part_ml, plan, table, stride, nh, nkv, dv, ldo, ps, ps_shift, num_pages,
+                         keep, sl2, softcap, slope_exp, sink, out_scale, dec_max, splits_max, DEC_PAGE_CAP, tickets, err);
 }
 
 }  // namespace
@@ -1156,29 +1167,35 @@ int launch_decode(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMa
 // Portions of many tokens on the tensor cores: 128 queries of two query heads per work item, the items
 // shared out among `ctas` CTAs (at most one per SM) by `work`, which xb_attn_prefill_work (host
 // library) makes from the step's portions: [ctas + 1] offsets, then (portion, query tile, first query
-// head, heads) per item, on the device.  `tokens` = rows of q.  Returns cudaErrorNotSupported (having done nothing)
-// for a head size over 128 or not a multiple of 16, or a page size that is no power of two >= 8.
+// head, heads) per item, on the device.  `tokens` = rows of q.  Queries and keys have d channels, values dv; a token's
+// outputs (nh x dv, times out_scale) start ldo elements apart.  `keep` > 0 beside a sliding window: the sequence's first
+// positions stay visible.  `sink` (float32 per head, nullable): one more entry of every softmax, of that score, without
+// a value.  Returns cudaErrorNotSupported (having done nothing) for a head size over 128 or not a multiple of 16, an
+// ldo that is no multiple of 8, or a page size that is no power of two >= 8.
 XB_EXPORT int xb_attn_prefill_tc(void* out, const void* q, const void* kc, const void* vc, const int* q_start,
                                  const int* start_pos, const int* table, int stride, int tokens,
-                                 int nh, int nkv, int d, int ps, int num_pages, int window, float scale, float softcap,
-                                 float slope_exp, const int* work, int ctas, int* err, cudaStream_t stream) {
+                                 int nh, int nkv, int d, int dv, long long ldo, int ps, int num_pages, int window, int keep,
+                                 float scale, float softcap, float slope_exp, const float* sink, float out_scale,
+                                 const int* work, int ctas, int* err, cudaStream_t stream) {
     if (ctas <= 0) return 0;
     int shift = -1;
     for (int s = 3; s < 20; ++s)
         if ((1 << s) == ps) shift = s;
-    if (d % 16 || d > 128 || d < 16 || nh % nkv || shift < 0 || !work) return (int)cudaErrorNotSupported;
-    CUtensorMap mq, mk, mv, mo;   // out has the layout of q; a warp stores its 32 rows
+    if (d % 16 || d > 128 || d < 16 || dv % 16 || dv > 128 || dv < 16 || ldo % 8 || ((uintptr_t)out & 15) || nh % nkv ||
+        shift < 0 || !work || (keep > 0 && window <= 0))
+        return (int)cudaErrorNotSupported;
+    CUtensorMap mq, mk, mv, mo;   // a warp stores its 32 rows
     const long long rows = (long long)num_pages * nkv * ps;
     const int box_rows = ps < KT ? ps : KT;
-    if (!map_q3(&mq, q, tokens, nh, d, 1, QT) || !map_q3(&mo, out, tokens, nh, d, 1, 32) || !map_rows(&mk, kc, rows, d, box_rows) ||
-        !map_rows(&mv, vc, rows, d, box_rows))
+    if (!map_q3(&mq, q, tokens, nh, d, (long long)nh * d, 1, QT) || !map_q3(&mo, out, tokens, nh, dv, ldo, 1, 32) ||
+        !map_rows(&mk, kc, rows, d, box_rows) || !map_rows(&mv, vc, rows, dv, box_rows))
         return (int)cudaErrorNotSupported;
     const float sl2 = scale * 1.4426950408889634f;
-    if (d <= 64)
-        return launch_prefill<64>(mq, mk, mv, mo, out, q_start, start_pos, table, stride, nh, nkv, d, ps, shift, num_pages, window,
-                                  sl2, softcap, slope_exp, work, ctas, err, stream);
-    return launch_prefill<128>(mq, mk, mv, mo, out, q_start, start_pos, table, stride, nh, nkv, d, ps, shift, num_pages, window,
-                               sl2, softcap, slope_exp, work, ctas, err, stream);
+    if (d <= 64 && dv <= 64)
+        return launch_prefill<64>(mq, mk, mv, mo, out, q_start, start_pos, table, stride, nh, nkv, dv, ldo, ps, shift, num_pages,
+                                  window, keep, sl2, softcap, slope_exp, sink, out_scale, work, ctas, err, stream);
+    return launch_prefill<128>(mq, mk, mv, mo, out, q_start, start_pos, table, stride, nh, nkv, dv, ldo, ps, shift, num_pages,
+                               window, keep, sl2, softcap, slope_exp, sink, out_scale, work, ctas, err, stream);
 }
 // int32 a plan for `tokens` small tokens and `ctas` target CTAs must hold.
 XB_EXPORT long long xb_attn_decode_plan_size(int tokens, int ctas, int nkv) {
@@ -1192,20 +1209,21 @@ XB_EXPORT long long xb_attn_decode_plan_size(int tokens, int ctas, int nkv) {
 // the step that is launched with programmatic dependent launch: xb_attn_decode_tc reads the plan
 // before it waits for the kernel before it.
 XB_EXPORT int xb_attn_decode_plan(int* plan, const int* positions, const int* req_of_token, const int* q_start,
-                                  int num_entries, int window, int dec_max, int direct, int tokens, int min_keys, int ctas,
-                                  int nkv, int* err, cudaStream_t stream) {
+                                  int num_entries, int window, int keep, int dec_max, int direct, int tokens, int min_keys,
+                                  int ctas, int nkv, int* err, cudaStream_t stream) {
     if (tokens <= 0) return 0;
     if (tokens > PLAN_TOKENS_MAX) return (int)cudaErrorNotSupported;
-    if (min_keys <= 0 || min_keys % KT || ctas <= 0 || nkv <= 0) return (int)cudaErrorInvalidValue;
+    if (min_keys <= 0 || min_keys % KT || ctas <= 0 || nkv <= 0 || (keep > 0 && window <= 0)) return (int)cudaErrorInvalidValue;
     const int capacity = tokens + ctas / nkv + 2;
     attn_decode_plan_kernel<<<1, PLAN_THREADS, 0, stream>>>(plan, capacity, positions, req_of_token, q_start, num_entries, window,
-                                                           dec_max, direct, tokens, min_keys / KT, ctas, nkv, err);
+                                                           keep, dec_max, direct, tokens, min_keys / KT, ctas, nkv, err);
     return xb_launch_status();
 }
 
 // The step's small tokens on the tensor cores, shared out as `plan` says (made by
-// xb_attn_decode_plan with the same tokens, ctas and kv heads, for the same window).  A token and
-// head in several pieces is merged through scratch: part_o [tokens, nh, splits_max, d] float32,
+// xb_attn_decode_plan with the same tokens, ctas and kv heads, for the same window and keep).  `keep`, `sink`, dv,
+// ldo and out_scale as for xb_attn_prefill_tc.  A token and
+// head in several pieces is merged through scratch: part_o [tokens, nh, splits_max, dv] float32,
 // part_ml [tokens, nh, splits_max, 2] float32 and tickets [tokens * kv heads] int32, zero before the
 // first launch (the kernel leaves them zero); splits_max must be at least
 // min(ctas / kv heads + 1, longest context / min_keys + 1).  `q_rows` = rows of q.  `overlap` != 0
@@ -1214,27 +1232,32 @@ XB_EXPORT int xb_attn_decode_plan(int* plan, const int* positions, const int* re
 // Returns cudaErrorNotSupported (having done nothing) for a head size over 128 or not a multiple of
 // 16, a page size that is no power of two >= 8, or more than 16 query heads per key/value head.
 XB_EXPORT int xb_attn_decode_tc(void* out, float* part_o, float* part_ml, const void* q, const void* kc, const void* vc,
-                                const int* plan, const int* table, int stride, int q_rows, int nh, int nkv, int d, int ps,
-                                int num_pages, float scale, float softcap, float slope_exp, int dec_max, int splits_max,
-                                int tokens, int ctas, int* tickets, int overlap, int* err, cudaStream_t stream) {
+                                const int* plan, const int* table, int stride, int q_rows, int nh, int nkv, int d, int dv,
+                                long long ldo, int ps, int num_pages, int keep, float scale, float softcap, float slope_exp,
+                                const float* sink, float out_scale, int dec_max, int splits_max, int tokens, int ctas,
+                                int* tickets, int overlap, int* err, cudaStream_t stream) {
     if (tokens <= 0) return 0;
     int shift = -1;
     for (int s = 3; s < 20; ++s)
         if ((1 << s) == ps) shift = s;
-    if (d % 16 || d > 128 || d < 16 || nh % nkv || nh / nkv > DEC_ROWS || shift < 0 || tokens > PLAN_TOKENS_MAX)
+    if (d % 16 || d > 128 || d < 16 || dv % 16 || dv > 128 || dv < 16 || ldo % 8 || ((uintptr_t)out & 15) || nh % nkv ||
+        nh / nkv > DEC_ROWS || shift < 0 || tokens > PLAN_TOKENS_MAX)
         return (int)cudaErrorNotSupported;
     if (!plan || splits_max <= 0 || ctas <= 0) return (int)cudaErrorInvalidValue;
     if (splits_max > 1 && (!part_o || !part_ml || !tickets)) return (int)cudaErrorInvalidValue;
     CUtensorMap mq, mk, mv;
     const long long rows = (long long)num_pages * nkv * ps;
     const int box_rows = ps < KT ? ps : KT;
-    if (!map_q3(&mq, q, q_rows, nh, d, nh / nkv, 1) || !map_rows(&mk, kc, rows, d, box_rows) || !map_rows(&mv, vc, rows, d, box_rows))
+    if (!map_q3(&mq, q, q_rows, nh, d, (long long)nh * d, nh / nkv, 1) || !map_rows(&mk, kc, rows, d, box_rows) ||
+        !map_rows(&mv, vc, rows, dv, box_rows))
         return (int)cudaErrorNotSupported;
     const float sl2 = scale * 1.4426950408889634f;
     const int pieces = tokens + ctas / nkv + 2;   // the most the plan can hold
-    if (d <= 64)
-        return launch_decode<64>(mq, mk, mv, out, part_o, part_ml, plan, pieces, table, stride, nh, nkv, d, ps, shift, num_pages,
-                                 sl2, softcap, slope_exp, dec_max, splits_max, tickets, overlap, err, stream);
-    return launch_decode<128>(mq, mk, mv, out, part_o, part_ml, plan, pieces, table, stride, nh, nkv, d, ps, shift, num_pages,
-                              sl2, softcap, slope_exp, dec_max, splits_max, tickets, overlap, err, stream);
+    if (d <= 64 && dv <= 64)
+        return launch_decode<64>(mq, mk, mv, out, part_o, part_ml, plan, pieces, table, stride, nh, nkv, dv, ldo, ps, shift,
+                                 num_pages, keep, sl2, softcap, slope_exp, sink, out_scale, dec_max, splits_max, tickets, overlap,
+                                 err, stream);
+    return launch_decode<128>(mq, mk, mv, out, part_o, part_ml, plan, pieces, table, stride, nh, nkv, dv, ldo, ps, shift,
+                              num_pages, keep, sl2, softcap, slope_exp, sink, out_scale, dec_max, splits_max, tickets, overlap, err,
+                              stream);
 }

@@ -390,8 +390,8 @@ __global__ void attention_plain_kernel(
     const T* __restrict__ v_cache, int k_stride, int v_stride, const float* __restrict__ sink,
     const int* __restrict__ positions,
     const int* __restrict__ req_of_token, const int* __restrict__ block_table, int table_stride,
-    int nh, int nkv, int d, int dv, int page_size, int num_pages, int window, float scale, float softcap, float slope_exp,
-    int chunk, int* err) {
+    int nh, int nkv, int d, int dv, int page_size, int num_pages, int window, int keep, float scale, float softcap,
+    float slope_exp, int chunk, long long ldo, float out_scale, int* err) {
     const int t = blockIdx.x;
     const int lane = threadIdx.x & 31;
     const int h = blockIdx.y * (blockDim.x >> 5) + (threadIdx.x >> 5);
@@ -400,7 +400,7 @@ __global__ void attention_plain_kernel(
     const int pos = positions[t];
     const int b = req_of_token[t];
     if (b < 0) {  // padding token
-        T* o = out + ((size_t)t * nh + h) * dv;
+        T* o = out + (size_t)t * ldo + (size_t)h * dv;
         for (int i = lane; i < dv; i += 32) o[i] = from_f32<T>(0.f);
         return;
     }
@@ -421,7 +421,9 @@ __global__ void attention_plain_kernel(
     int lo = (window > 0 && pos - window + 1 > 0) ? pos - window + 1 : 0;
     if (chunk > 0) lo = max(lo, pos / chunk * chunk);
     const float slope = slope_exp > 0.f ? exp2f(-slope_exp * (float)(h + 1) / (float)nh) : 0.f;
-    for (int j = lo; j <= pos; ++j) {
+    const int kept = min(keep, lo);     // the sequence's first positions, where they stay visible beside a window
+    for (int n = 0; n < kept + pos - lo + 1; ++n) {
+        const int j = n < kept ? n : lo + n - kept;
         const int page = table[j / page_size];
         if (page < 0 || page >= num_pages) {
             if (lane == 0) atomicOr(err, XB_ERR_BAD_PAGE);
@@ -450,8 +452,8 @@ __global__ void attention_plain_kernel(
         }
         m = m_new;
     }
-    const float inv = l > 0.f ? 1.f / l : 0.f;
-    T* o = out + ((size_t)t * nh + h) * dv;
+    const float inv = l > 0.f ? out_scale / l : 0.f;
+    T* o = out + (size_t)t * ldo + (size_t)h * dv;
 #pragma unroll
     for (int e = 0; e < MAXE; ++e) {
         const int i = e * 32 + lane;
@@ -464,15 +466,16 @@ static int attention_plain_launch(void* out, const void* q, long long q_ts, long
                                   int k_stride, int v_stride, const float* sink,
                                   const int* positions, const int* req_of_token, const int* block_table,
                                   int table_stride, int tokens, int nh, int nkv, int d, int dv, int page_size,
-                                  int num_pages, int window, float scale, float softcap, float slope_exp, int chunk, int* err,
-                                  cudaStream_t stream) {
+                                  int num_pages, int window, int keep, float scale, float softcap, float slope_exp, int chunk,
+                                  long long ldo, float out_scale, int* err, cudaStream_t stream) {
     dim3 grid(tokens, (nh + 3) / 4);
     const int dm = d > dv ? d : dv;
 #define XB_ATT(MAXE)                                                                              \
     attention_plain_kernel<T, MAXE><<<grid, 128, 0, stream>>>(                                    \
         (T*)out, (const T*)q, q_ts, q_hs, (const T*)kc, (const T*)vc, k_stride, v_stride, sink,  \
         positions, req_of_token, block_table,                                                    \
-        table_stride, nh, nkv, d, dv, page_size, num_pages, window, scale, softcap, slope_exp, chunk, err)
+        table_stride, nh, nkv, d, dv, page_size, num_pages, window, keep, scale, softcap, slope_exp,      \
+        chunk, ldo, out_scale, err)
     if (dm <= 64) XB_ATT(2);
     else if (dm <= 128) XB_ATT(4);
     else if (dm <= 256) XB_ATT(8);
@@ -488,16 +491,16 @@ XB_EXPORT int xb_attention_plain(int dtype, void* out, const void* q, long long 
                                  const void* v_cache, int k_stride, int v_stride, const float* sink,
                                  const int* positions, const int* req_of_token,
                                  const int* block_table, int table_stride, int tokens, int nh, int nkv,
-                                 int d, int dv, int page_size, int num_pages, int window, float scale, float softcap,
-                                 float slope_exp, int chunk, int* err, cudaStream_t stream) {
+                                 int d, int dv, int page_size, int num_pages, int window, int keep, float scale, float softcap,
+                                 float slope_exp, int chunk, long long ldo, float out_scale, int* err, cudaStream_t stream) {
     if (tokens <= 0) return 0;
     if (dtype == XB_F32)
         return attention_plain_launch<float>(out, q, q_ts, q_hs, k_cache, v_cache, k_stride, v_stride, sink, positions,
                                              req_of_token, block_table,
-                                             table_stride, tokens, nh, nkv, d, dv, page_size, num_pages, window, scale, softcap, slope_exp, chunk, err, stream);
+                                             table_stride, tokens, nh, nkv, d, dv, page_size, num_pages, window, keep, scale, softcap, slope_exp, chunk, ldo, out_scale, err, stream);
     return attention_plain_launch<__nv_bfloat16>(out, q, q_ts, q_hs, k_cache, v_cache, k_stride, v_stride, sink, positions,
                                                  req_of_token, block_table,
-                                                 table_stride, tokens, nh, nkv, d, dv, page_size, num_pages, window, scale, softcap, slope_exp, chunk, err, stream);
+                                                 table_stride, tokens, nh, nkv, d, dv, page_size, num_pages, window, keep, scale, softcap, slope_exp, chunk, ldo, out_scale, err, stream);
 }
 
 // ------------------------------------------------------------------------------------------

@@ -16,7 +16,7 @@ using namespace xb;
 
 // ---- cache manager -------------------------------------------------------------------------
 XB_API void* xb_cm_create(int n_groups, const int* page_sizes, const int* num_pages, const int* windows,
-                          int max_requests) {
+                          const int* keep_first, int max_requests) {
     if (n_groups <= 0 || max_requests <= 0) return nullptr;
     std::vector<GroupSpec> groups(n_groups);
     for (int g = 0; g < n_groups; ++g) {
@@ -24,6 +24,7 @@ XB_API void* xb_cm_create(int n_groups, const int* page_sizes, const int* num_pa
         groups[g].page_size = page_sizes[g];
         groups[g].num_pages = num_pages[g];
         groups[g].window = windows[g];
+        groups[g].keep_first = keep_first ? keep_first[g] : 0;
     }
     return new CacheManager(groups, max_requests);
 }
@@ -162,8 +163,9 @@ XB_API long long xb_assemble(void* h, int B, const int* slots, const int* counts
 // one head where two-head items would leave CTAs idle (short portions, few heads), two otherwise.
 // out: [ctas + 1] offsets (in items) then 4 int32 per item: portion, query tile, first query head, heads.
 // Returns the number of int32 written (-1: capacity too small) and the number of CTAs in *ctas_out.
+// keep_first > 0 (beside a sliding window): the key tiles of the sequence's first keep_first positions count too.
 XB_API long long xb_attn_prefill_work(int B, const int* counts, const int* starts, int dec_max, int window,
-                                      int heads, int kv_heads, int max_ctas, int32_t* out, long long capacity,
+                                      int keep_first, int heads, int kv_heads, int max_ctas, int32_t* out, long long capacity,
                                       int* ctas_out) {
     // costs in sixths of a key tile of two heads: a tile of one head takes about two thirds of the time of a tile
     // of two (measured at long contexts: 0.76 us against 1.15 us), an item's start about three tiles
@@ -178,7 +180,8 @@ XB_API long long xb_attn_prefill_work(int B, const int* counts, const int* start
             // window > 0: a sliding window; window < 0: chunks of -window positions counted from position 0
             const int last_key = p0 + rows - 1;
             const int first_key = window > 0 ? std::max(0, p0 - window + 1) : (window < 0 ? p0 / (-window) * (-window) : 0);
-            tiles.push_back({last_key / KT - first_key / KT + 1, b, ti});
+            const int kept = window > 0 && keep_first > 0 ? std::min((keep_first + KT - 1) / KT, first_key / KT) : 0;
+            tiles.push_back({kept + last_key / KT - first_key / KT + 1, b, ti});
         }
     }
     *ctas_out = 0;

@@ -75,6 +75,12 @@ int CacheManager::first_needed_page(int g, int len) const {
     return first_key > 0 ? first_key / s.page_size : 0;
 }
 
+// Pages at a sequence's start that a windowed group never gives back while the request lives.
+int CacheManager::kept_pages(int g) const {
+    const GroupSpec& s = groups_[g];
+    return s.window > 0 && s.keep_first > 0 ? (s.keep_first + s.page_size - 1) / s.page_size : 0;
+}
+
 int CacheManager::pages_needed(int slot, int new_len, int g) const {
     if (!is_live(slot)) return -1;
     const Request& r = reqs_[slot];
@@ -112,7 +118,7 @@ bool CacheManager::advance(int slot, int new_len) {
     r.len = new_len;
     for (int g = 0; g < (int)groups_.size(); ++g) {
         const int keep_from = std::min(first_needed_page(g, new_len), (int)r.tables[g].size());
-        for (int i = 0; i < keep_from; ++i) {
+        for (int i = kept_pages(g); i < keep_from; ++i) {
             if (r.tables[g][i] >= 0) {
                 if (pools_[g].give(r.tables[g][i]) && log_freed_) freed_.emplace_back(g, r.tables[g][i]);
                 r.tables[g][i] = -1;

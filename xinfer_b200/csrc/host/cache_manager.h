@@ -19,6 +19,7 @@ struct GroupSpec {
     int page_size = 16;
     int num_pages = 0;
     int window = 0;  // <= 0: every earlier key is kept; else a query at p reads keys > p - window
+    int keep_first = 0;  // beside a window: keys at positions below this are read by every query
 };
 
 // A pool of page ids, reused first-in first-out so that tests can predict which page comes next.
@@ -82,6 +83,7 @@ private:
         std::vector<std::vector<int32_t>> tables;  // per group, indexed by position / page_size
     };
     int first_needed_page(int g, int len) const;
+    int kept_pages(int g) const;
     bool log_freed_ = false;
     std::vector<std::pair<int32_t, int32_t>> freed_;
 

@@ -20,9 +20,10 @@ AddStatus Scheduler::add(int64_t req_id, const int32_t* prompt, int n, int max_t
         const GroupSpec& s = cache_->group(g);
         int most = total;
         if (s.window > 0) {
-            // a windowed group holds at most one portion plus the window behind it
+            // a windowed group holds at most one portion, the window behind it and the first positions it keeps
             const int portion = std::min(std::min(cfg_.prefill_chunk_size, cfg_.max_num_batched_tokens), n);
-            most = std::min(total, s.window + portion + s.page_size);
+            const int kept = s.keep_first > 0 ? (s.keep_first + s.page_size - 1) / s.page_size * s.page_size : 0;
+            most = (int)std::min<long long>(total, (long long)s.window + portion + s.page_size + kept);
         }
         if ((most + s.page_size - 1) / s.page_size > s.num_pages) return ADD_NEVER_FITS;
     }

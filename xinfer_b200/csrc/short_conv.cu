@@ -138,7 +138,8 @@ __global__ void __launch_bounds__(128) conv_silu_run_kernel(TO* __restrict__ y, 
     }
 }
 
-__global__ void conv_state_kernel(float* __restrict__ state, const float* __restrict__ u, long long u_ld, int u_off,
+template <typename T>
+__global__ void conv_state_kernel(T* __restrict__ state, const T* __restrict__ u, long long u_ld, int u_off,
                                   const int* __restrict__ q_start, const int* __restrict__ slots, int C, int K) {
     const int b = blockIdx.y;
     const int c = blockIdx.x * blockDim.x + threadIdx.x;
@@ -146,8 +147,8 @@ __global__ void conv_state_kernel(float* __restrict__ state, const float* __rest
     if (c >= C || slot < 0) return;
     const int t0 = q_start[b], n = q_start[b + 1] - t0;
     if (n <= 0) return;
-    float keep[SC_MAX_TAPS];
-    float* st = state + (size_t)slot * (K - 1) * C + c;
+    T keep[SC_MAX_TAPS];
+    T* st = state + (size_t)slot * (K - 1) * C + c;
 #pragma unroll
     for (int k = 0; k < SC_MAX_TAPS; ++k) {
         if (k >= K - 1) break;
@@ -210,11 +211,15 @@ XB_EXPORT int xb_conv_silu(int out_dtype, void* y, const float* u, long long u_l
     return xb_launch_status();
 }
 
-XB_EXPORT int xb_conv_state(float* state, const float* u, long long u_ld, int u_off, const int* q_start, const int* slots,
+XB_EXPORT int xb_conv_state(int dtype, void* state, const void* u, long long u_ld, int u_off, const int* q_start, const int* slots,
                             int entries, int C, int K, cudaStream_t stream) {
     if (entries <= 0 || C <= 0 || K <= 1) return 0;
     if (K > SC_MAX_TAPS) return (int)cudaErrorInvalidValue;
     const dim3 grid((C + 127) / 128, entries);
-    conv_state_kernel<<<grid, 128, 0, stream>>>(state, u, u_ld, u_off, q_start, slots, C, K);
+    if (dtype == XB_F32)
+        conv_state_kernel<float><<<grid, 128, 0, stream>>>((float*)state, (const float*)u, u_ld, u_off, q_start, slots, C, K);
+    else
+        conv_state_kernel<__nv_bfloat16><<<grid, 128, 0, stream>>>((__nv_bfloat16*)state, (const __nv_bfloat16*)u, u_ld, u_off,
+                                                                   q_start, slots, C, K);
     return xb_launch_status();
 }

@@ -4,6 +4,8 @@
 //   delta_rule_kernel       (gated delta rule)      S[d, dv]: S <- diag(g) S,  u = beta (v - S^T k),  S <- S + k u^T,
 //                                                             o = S^T q      (read after the token's own update)    
 //   linear_scan_kernel      (gated linear attention)  S[d, dv]: S <- diag(alpha) S + k v^T,  o = scale S^T q
+//   matrix_memory_kernel    (xLSTM's mLSTM)         S[d, dv]: S <- e^(f+m-m') S + e^(i-m') k v^T, n[d] likewise with k alone,
+//                                                             o = S^T q and the divisor max(|n . q|, e^(-m')) + eps
 //   low_rank_decay_kernel   alpha = sigmoid(W_a2 low + b)^(1 / tau) for it, per token and key channel
 //   gated_head_norm_kernel  the gate and the RMS norm over a head (or a group of channels) behind either
 //
@@ -473,6 +475,191 @@ __global__ void __launch_bounds__(384, 1) linear_scan_kernel(float* __restrict__
     }
 }
 
+// proj[t] holds q (H*d from column 0), k (H*d behind it), v (H*dv behind that) and at gate_off the input gates' and the
+// forget gates' pre-activations (H each, without their biases).  With i = cap tanh((z_i + b_i) / cap) and
+// f = -softplus(-cap tanh((z_f + b_f) / cap)):
+//   m' = max(f + m, i);  a = e^(f + m - m');  b = e^(i - m');   S <- a S + b k v^T;   n <- a n + b k
+//   o[t, h*dv ..] = scale S^T q,   div[t, h] = max(|scale n . q|, e^(-m')) + div_eps          after the token's own write
+// state_s [slots, H, d, dv], state_n [slots, H, d].  The running maximum m is read by every block of a head but left by
+// one of them, so it has two places: state_m [slots, H, 2, 2] holds (tokens it stands behind, m) twice; a step reads the
+// place that stands behind its start and writes the other one.  Zeros are a request's start.
+// Shared memory: two stages of q[TT][DP] k[TT][DP] v[TT][VT] a[TT] b[TT] e^(-m')[TT], then two tiles o[TT][VT].  Besides
+// the computing and the feeding warps there is one (warp `cw`) that carries n where the block has the head's first
+// columns; the first feeding warp works out the gates, a lane per token, and walks m over the tile.
+template <int DS>
+__global__ void __launch_bounds__(384, 1) matrix_memory_kernel(
+    float* __restrict__ o, float* __restrict__ div, const float* __restrict__ proj, long long ldp, int gate_off,
+    const float* __restrict__ bi, const float* __restrict__ bf, float cap, float* __restrict__ state_s,
+    float* __restrict__ state_n, float* state_m, const int* __restrict__ q_start, const int* __restrict__ start_pos,
+    const int* __restrict__ slots, int H, int d, int dv, float scale, float div_eps, int TT, int stage, int cw, int vec) {
+    extern __shared__ __align__(16) float scan_smem[];
+    constexpr int CGW = 32 / DS, DP = DS * kRowsPad, NR = DS * kRows;
+    const int b = blockIdx.x, h = blockIdx.y;
+    const int lane = threadIdx.x & 31, w = threadIdx.x >> 5;
+    const int VT = cw * CGW * 2, c_base = blockIdx.z * VT;
+    const int slot = slots[b];
+    const int t0 = q_start[b], t1 = q_start[b + 1];
+    if (slot < 0 || t1 <= t0) return;
+    const int ntiles = (t1 - t0 + TT - 1) / TT;
+    float* so = scan_smem + 2 * stage;
+    if (w > cw) {
+        // feeding warps: warp `pi` of `pw` takes tokens pi, pi + pw, ... of every tile
+        const int pi = w - cw - 1, pw = (blockDim.x >> 5) - cw - 1;
+        float* place = state_m + ((size_t)slot * H + h) * 4;
+        const float at_start = (float)start_pos[b];
+        const int from = place[0] == at_start ? 0 : 1;
+        float m = place[2 * from + 1];
+        const float b_i = bi[h], b_f = bf[h];
+        auto bring = [&](int tile) {
+            float* sq = scan_smem + (tile & 1) * stage;
+            float* sk = sq + TT * DP;
+            float* sv = sk + TT * DP;
+            float* sg = sv + TT * VT;
+            const int tb = t0 + tile * TT, nt = min(TT, t1 - tb);
+            float zi = 0.f, zf = 0.f;
+            if (pi == 0 && lane < nt) {
+                const float* g = proj + (size_t)(tb + lane) * ldp + gate_off + h;
+                zi = g[0];
+                zf = g[H];
+            }
+            for (int tt = pi; tt < nt; tt += pw) {
+                const float* row = proj + (size_t)(tb + tt) * ldp;
+                stage_rows(sq + tt * DP, row + h * d, d, NR, lane, vec);
+                stage_rows(sk + tt * DP, row + (H + h) * d, d, NR, lane, vec);
+                stage_cols(sv + tt * VT, row + 2 * H * d + h * dv, c_base, dv, VT, lane, vec);
+            }
+            if (pi == 0) {
+                const float gi = cap * tanhf((zi + b_i) / cap), y = cap * tanhf((zf + b_f) / cap);
+                const float gf = fminf(y, 0.f) - log1pf(expf(-fabsf(y)));      // log of the sigmoid
+                float before = m, after = m;
+                for (int tt = 0; tt < nt; ++tt) {
+                    const float f_t = __shfl_sync(0xffffffffu, gf, tt), i_t = __shfl_sync(0xffffffffu, gi, tt);
+                    const float next = fmaxf(f_t + m, i_t);
+                    if (lane == tt) {
+                        before = m;
+                        after = next;
+                    }
+                    m = next;
+                }
+                if (lane < nt) {
+                    sg[lane] = expf(gf + before - after);
+                    sg[TT + lane] = expf(gi - after);
+                    sg[2 * TT + lane] = expf(-after);
+                }
+            }
+            scan_cp_land();
+        };
+        auto leave = [&](int tile) {
+            const float* src = so + (tile & 1) * TT * VT;
+            const int tb = t0 + tile * TT, nt = min(TT, t1 - tb);
+            for (int tt = pi; tt < nt; tt += pw)
+                for (int c = lane; c < VT; c += 32)
+                    if (c_base + c < dv) o[((size_t)(tb + tt) * H + h) * dv + c_base + c] = src[tt * VT + c];
+        };
+        bring(0);
+        __syncthreads();
+        for (int tile = 0; tile < ntiles; ++tile) {
+            if (tile + 1 < ntiles) bring(tile + 1);
+            if (tile > 0) leave(tile - 1);
+            __syncthreads();
+        }
+        leave(ntiles - 1);
+        if (pi == 0 && lane == 0 && blockIdx.z == 0) {
+            place[2 * (from ^ 1)] = at_start + (float)(t1 - t0);
+            place[2 * (from ^ 1) + 1] = m;
+        }
+        return;
+    }
+    if (w == cw) {
+        // n and the divisors; a lane keeps rows lane, lane + 32, ...
+        constexpr int NN = (NR + 31) / 32;
+        const bool mine = blockIdx.z == 0;
+        float n[NN];
+        float* sn = state_n + ((size_t)slot * H + h) * d;
+#pragma unroll
+        for (int r = 0; r < NN; ++r) n[r] = mine && lane + 32 * r < d ? sn[lane + 32 * r] : 0.f;
+        __syncthreads();
+        for (int tile = 0; tile < ntiles; ++tile) {
+            if (mine) {
+                const float* sq = scan_smem + (tile & 1) * stage;
+                const float* sk = sq + TT * DP;
+                const float* sg = scan_smem + (tile & 1) * stage + 2 * TT * DP + TT * VT;
+                const int nt = min(TT, t1 - t0 - tile * TT);
+                float* dst = div + (size_t)(t0 + tile * TT) * H + h;
+#pragma unroll 4
+                for (int tt = 0; tt < nt; ++tt) {
+                    const float a = sg[tt], bb = sg[TT + tt];
+                    float acc = 0.f;
+#pragma unroll
+                    for (int r = 0; r < NN; ++r) {
+                        if (lane + 32 * r >= NR) break;
+                        const int at = tt * DP + padded_row(lane + 32 * r);
+                        n[r] = fmaf(a, n[r], bb * sk[at]);
+                        acc = fmaf(n[r], sq[at], acc);
+                    }
+                    acc = warp_total(acc);
+                    if (lane == 0) dst[(size_t)tt * H] = fmaxf(fabsf(scale * acc), sg[2 * TT + tt]) + div_eps;
+                }
+            }
+            __syncthreads();
+        }
+#pragma unroll
+        for (int r = 0; r < NN; ++r)
+            if (mine && lane + 32 * r < d) sn[lane + 32 * r] = n[r];
+        return;
+    }
+    const int ds = lane / CGW, cl = (w * CGW + lane % CGW) * 2, v0 = c_base + cl;
+    float S0[kRows], S1[kRows];
+    float* st = state_s + ((size_t)slot * H + h) * d * dv;
+#pragma unroll
+    for (int r = 0; r < kRows; ++r) {
+        const int j = ds * kRows + r;
+        S0[r] = (j < d && v0 < dv) ? st[(size_t)j * dv + v0] : 0.f;
+        S1[r] = (j < d && v0 + 1 < dv) ? st[(size_t)j * dv + v0 + 1] : 0.f;
+    }
+    __syncthreads();
+    for (int tile = 0; tile < ntiles; ++tile) {
+        const float* sq = scan_smem + (tile & 1) * stage + ds * kRowsPad;
+        const float* sk = sq + TT * DP;
+        const float* sv = scan_smem + (tile & 1) * stage + 2 * TT * DP;
+        const float* sg = sv + TT * VT;
+        sv += cl;
+        float* out = so + (tile & 1) * TT * VT + cl;
+        const int nt = min(TT, t1 - t0 - tile * TT);
+        for (int tt = 0; tt < nt; ++tt, sq += DP, sk += DP, sv += VT, out += VT) {
+            const float dec = sg[tt], in = sg[TT + tt];
+            const float2 vv = *reinterpret_cast<const float2*>(sv);
+            const float w0 = in * vv.x, w1 = in * vv.y;
+            const float4* qp = reinterpret_cast<const float4*>(sq);
+            const float4* kp = reinterpret_cast<const float4*>(sk);
+            float a0 = 0.f, a1 = 0.f;
+#pragma unroll
+            for (int i = 0; i < kRows / 4; ++i) {
+                const float4 q4 = qp[i], k4 = kp[i];
+                const float qq[4] = {q4.x, q4.y, q4.z, q4.w}, kq[4] = {k4.x, k4.y, k4.z, k4.w};
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                    const int r = 4 * i + e;
+                    S0[r] = fmaf(dec, S0[r], kq[e] * w0);
+                    S1[r] = fmaf(dec, S1[r], kq[e] * w1);
+                    a0 = fmaf(S0[r], qq[e], a0);
+                    a1 = fmaf(S1[r], qq[e], a1);
+                }
+            }
+            a0 = fold_rows<DS>(a0);
+            a1 = fold_rows<DS>(a1);
+            if (ds == 0) *reinterpret_cast<float2*>(out) = make_float2(scale * a0, scale * a1);
+        }
+        __syncthreads();
+    }
+#pragma unroll
+    for (int r = 0; r < kRows; ++r) {
+        const int j = ds * kRows + r;
+        if (j < d && v0 < dv) st[(size_t)j * dv + v0] = S0[r];
+        if (j < d && v0 + 1 < dv) st[(size_t)j * dv + v0 + 1] = S1[r];
+    }
+}
+
 // alpha[t, c] = sigmoid(z)^(1 / tau) = exp(-softplus(-z) / tau),  z = bias[c] + sum_r w[c, r] low[t, r].  low is a
 // column range of wider float32 rows.  A block takes a tile of tokens and 128 channels, a thread one channel of all its
 // tokens; both operands pass through shared memory, so that memory is read in order; r in order for every output.
@@ -542,11 +729,11 @@ static inline int scan_warps(int cols, int ds, long long heads_total) {
 
 static inline bool scan_aligned16(const void* p) { return ((uintptr_t)p & 15) == 0; }
 
-// Floats of one stage (`vectors` row vectors and two scalars per token beside the column tile), rounded so that
+// Floats of one stage (`vectors` row vectors and a few scalars per token beside the column tile), rounded so that
 // the second stage stays 16-byte aligned; the tile shrinks until two stages and two output tiles fit.
-static inline void scan_tile(int vectors, int ds, int vt, int& tt, int& stage, size_t& bytes) {
+static inline void scan_tile(int vectors, int ds, int vt, int& tt, int& stage, size_t& bytes, int scalars = 2) {
     for (tt = kScanTile;; tt /= 2) {
-        stage = (tt * (vectors * ds * kRowsPad + vt + 2) + 3) & ~3;
+        stage = (tt * (vectors * ds * kRowsPad + vt + scalars) + 3) & ~3;
         bytes = ((size_t)2 * stage + (size_t)2 * tt * vt) * sizeof(float);
         if (bytes <= 200 * 1024 || tt == 1) return;
     }
@@ -631,6 +818,26 @@ XB_EXPORT int xb_linear_scan(float* o, const float* proj, long long ldp, const f
     return xb_launch_status();
 }
 
+XB_EXPORT int xb_matrix_memory(float* o, float* div, const float* proj, long long ldp, int gate_off, const float* bi,
+                               const float* bf, float cap, float* state_s, float* state_n, float* state_m, const int* q_start,
+                               const int* start_pos, const int* slots, int entries, int H, int d, int dv, float scale,
+                               float div_eps, cudaStream_t stream) {
+    if (entries <= 0) return 0;
+    if (d < 1 || d > 32 * kRows || dv < 1 || H < 1 || H > 65535 || !(cap > 0.f)) return (int)cudaErrorInvalidValue;
+    const int ds = scan_row_groups(d);
+    const int warps = scan_warps(dv, ds, (long long)entries * H);
+    const int vt = warps * (32 / ds) * 2;
+    int tt, stage;
+    size_t bytes;
+    scan_tile(2, ds, vt, tt, stage, bytes, 3);
+    const dim3 grid(entries, H, (dv + vt - 1) / vt);
+    const int threads = (warps + 1 + (warps == 8 ? 3 : 4)) * 32;   // the warp of n, then three or four feeding warps
+    const int vec = scan_aligned16(proj) && ldp % 4 == 0 && d % 4 == 0 && dv % 4 == 0 && vt % 4 == 0;
+    XB_SCAN_DISPATCH(matrix_memory_kernel, ds, o, div, proj, ldp, gate_off, bi, bf, cap, state_s, state_n, state_m, q_start,
+                     start_pos, slots, H, d, dv, scale, div_eps, tt, stage, warps, vec)
+    return xb_launch_status();
+}
+
 XB_EXPORT int xb_low_rank_decay(float* alpha, const float* low, long long ldl, const float* w, const float* bias, int tokens,
                                 int C, int R, float tau, cudaStream_t stream) {
     if (tokens <= 0 || C <= 0) return 0;
@@ -645,18 +852,21 @@ XB_EXPORT int xb_low_rank_decay(float* alpha, const float* low, long long ldl, c
 //   mode 0:  v = y * silu(gate);  out = v * rsqrt(mean(v^2) + eps) * w[c mod w_len]          (gate before the norm)
 //   mode 1:  out = y * rsqrt(mean(y^2) + eps) * w[c mod w_len] * sigmoid(gate)               (gate behind it)
 //   mode 2:  the same with silu(gate)
-// gate is column g_off + c of a wider float32 row.
+// gate is column g_off + c of a wider float32 row.  div (nullable): every y of a part is first divided by div[t, part].
+// out's rows lie ldo apart and receive out_scale times the result.
 template <typename TO>
 __global__ void gated_head_norm_kernel(TO* __restrict__ out, const float* __restrict__ y, const float* __restrict__ gate,
                                        long long ldg, int g_off, const float* __restrict__ w, int w_len, int W, int part,
-                                       float eps, int mode) {
+                                       float eps, int mode, const float* __restrict__ div, long long ldo, float out_scale) {
     __shared__ float scratch[33];
     const int t = blockIdx.x, c0 = blockIdx.y * part;
     const float* yr = y + (size_t)t * W + c0;
     const float* gr = gate + (size_t)t * ldg + g_off + c0;
+    float dv = div ? div[(size_t)t * gridDim.y + blockIdx.y] : 1.f;
+    if (dv == 0.f) dv = 1.f;        // (a padding token's, which nothing has written)
     float ss = 0.f;
     for (int i = threadIdx.x; i < part; i += blockDim.x) {
-        float v = yr[i];
+        float v = yr[i] / dv;
         if (mode == 0) {
             const float z = gr[i];
             v *= z / (1.f + expf(-z));
@@ -664,15 +874,15 @@ __global__ void gated_head_norm_kernel(TO* __restrict__ out, const float* __rest
         ss = fmaf(v, v, ss);
     }
     const float inv = 1.f / sqrtf(block_sum(ss, scratch) / (float)part + eps);
-    TO* o = out + (size_t)t * W + c0;
+    TO* o = out + (size_t)t * ldo + c0;
     for (int i = threadIdx.x; i < part; i += blockDim.x) {
         const float z = gr[i];
-        float v = yr[i];
+        float v = yr[i] / dv;
         if (mode == 0)
             v = v * (z / (1.f + expf(-z))) * inv * w[(c0 + i) % w_len];
         else
             v = v * inv * w[(c0 + i) % w_len] * (mode == 2 ? z * sigmoid_exact(z) : sigmoid_exact(z));
-        o[i] = from_f32<TO>(v);
+        o[i] = from_f32<TO>(out_scale * v);
     }
 }
 
@@ -682,7 +892,8 @@ template <typename TO, int NV>
 __global__ void __launch_bounds__(256) gated_head_norm_warp_kernel(TO* __restrict__ out, const float* __restrict__ y,
                                                                    const float* __restrict__ gate, long long ldg, int g_off,
                                                                    const float* __restrict__ w, int w_len, int W, int part,
-                                                                   float eps, int mode, long long units) {
+                                                                   float eps, int mode, const float* __restrict__ div,
+                                                                   long long ldo, float out_scale, long long units) {
     const int lane = threadIdx.x & 31;
     const long long unit = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
     if (unit >= units) return;
@@ -692,36 +903,40 @@ __global__ void __launch_bounds__(256) gated_head_norm_warp_kernel(TO* __restric
     const float* yr = y + (size_t)t * W + c0;
     const float* gr = gate + (size_t)t * ldg + g_off + c0;
     float v[NV], z[NV];
+    float dv = div ? div[unit] : 1.f;
+    if (dv == 0.f) dv = 1.f;        // (a padding token's, which nothing has written)
     float ss = 0.f;
 #pragma unroll
     for (int k = 0; k < NV; ++k) {
         const int i = lane + 32 * k;
         v[k] = i < part ? yr[i] : 0.f;
         z[k] = i < part ? gr[i] : 0.f;
+        if (div) v[k] /= dv;
         if (mode == 0) v[k] *= z[k] / (1.f + expf(-z[k]));
         ss = fmaf(v[k], v[k], ss);
     }
     const float inv = 1.f / sqrtf(warp_total(ss) / (float)part + eps);
-    TO* o = out + (size_t)t * W + c0;
+    TO* o = out + (size_t)t * ldo + c0;
 #pragma unroll
     for (int k = 0; k < NV; ++k) {
         const int i = lane + 32 * k;
         if (i >= part) continue;
         float r = v[k] * inv * w[(c0 + i) % w_len];
         if (mode != 0) r *= mode == 2 ? z[k] * sigmoid_exact(z[k]) : sigmoid_exact(z[k]);
-        o[i] = from_f32<TO>(r);
+        o[i] = from_f32<TO>(out_scale * r);
     }
 }
 
 template <typename TO>
 static void gated_head_norm_launch(TO* out, const float* y, const float* gate, long long ldg, int g_off, const float* w,
-                                   int w_len, int tokens, int W, int part, float eps, int mode, cudaStream_t stream) {
+                                   int w_len, int tokens, int W, int part, float eps, int mode, const float* div,
+                                   long long ldo, float out_scale, cudaStream_t stream) {
     const long long units = (long long)tokens * (W / part);
     const int warps = 8;
     const unsigned blocks = (unsigned)((units + warps - 1) / warps);
 #define XB_HEAD_NORM_NV(NVV)                                                                                              \
     gated_head_norm_warp_kernel<TO, NVV><<<blocks, warps * 32, 0, stream>>>(out, y, gate, ldg, g_off, w, w_len, W, part, \
-                                                                            eps, mode, units)
+                                                                            eps, mode, div, ldo, out_scale, units)
     if (part <= 32) XB_HEAD_NORM_NV(1);
     else if (part <= 64) XB_HEAD_NORM_NV(2);
     else if (part <= 128) XB_HEAD_NORM_NV(4);
@@ -730,20 +945,22 @@ static void gated_head_norm_launch(TO* out, const float* y, const float* gate, l
     else {
         const dim3 grid(tokens, W / part);
         const int threads = part >= 1024 ? 256 : 128;
-        gated_head_norm_kernel<TO><<<grid, threads, 0, stream>>>(out, y, gate, ldg, g_off, w, w_len, W, part, eps, mode);
+        gated_head_norm_kernel<TO><<<grid, threads, 0, stream>>>(out, y, gate, ldg, g_off, w, w_len, W, part, eps, mode, div, ldo,
+                                                             out_scale);
     }
 #undef XB_HEAD_NORM_NV
 }
 
 XB_EXPORT int xb_gated_head_norm(int out_dtype, void* out, const float* y, const float* gate, long long ldg, int g_off,
                                  const float* w, int w_len, int tokens, int W, int part, float eps, int mode,
-                                 cudaStream_t stream) {
+                                 const float* div, long long ldo, float out_scale, cudaStream_t stream) {
     if (tokens <= 0 || W <= 0) return 0;
     if (part <= 0 || W % part || W / part > 65535) return (int)cudaErrorInvalidValue;
     if (out_dtype == XB_F32)
-        gated_head_norm_launch<float>((float*)out, y, gate, ldg, g_off, w, w_len, tokens, W, part, eps, mode, stream);
+        gated_head_norm_launch<float>((float*)out, y, gate, ldg, g_off, w, w_len, tokens, W, part, eps, mode, div, ldo,
+                                      out_scale, stream);
     else
         gated_head_norm_launch<__nv_bfloat16>((__nv_bfloat16*)out, y, gate, ldg, g_off, w, w_len, tokens, W, part, eps, mode,
-                                              stream);
+                                              div, ldo, out_scale, stream);
     return xb_launch_status();
 }

@@ -25,6 +25,11 @@
 // projected, before norm and rotation, double as values; the bias is read at the same offset).
 // `bias` (float32, laid out like a qkv row; absent: none) is added to q, k and v first.  With temp_every > 0 a
 // query at position p is multiplied, last of all, by 1 + temp_coef * ln(floor((p + 1) / temp_every) + 1).
+// With CONV every channel of the row first passes a causal convolution over time, y_t = sum_j taps[j, c] u_(t-K+1+j),c
+// (taps [K, channels], no bias): the K-1 rows before a step's first token of a request come from conv_state[slot]
+// ([K-1, channels], oldest first, in the rows' own type), the others from the rows of this step.  keep_state: every
+// request brings one token, and the block that has read its old rows leaves the last K-1 there.
+// value_eps >= 0: a value head is divided by its root mean square (this eps under the root) before it is cached.
 // q goes to q_out[t, h], k and v into their pages ([page, kv_head, slot, d] and [.., dv]).
 // One block per token, one warp per head at a time; the angles' cos/sin are formed once per token.
 // ------------------------------------------------------------------------------------------
@@ -57,7 +62,7 @@ __device__ __forceinline__ void store4<__nv_bfloat16>(__nv_bfloat16* p, const fl
     *reinterpret_cast<uint2*>(p) = t;
 }
 
-template <typename T>
+template <typename T, bool CONV>
 __global__ void qkv_prepare_kernel(T* __restrict__ q_out, T* __restrict__ k_cache, T* __restrict__ v_cache,
                                    const T* __restrict__ qkv, const float* __restrict__ q_w, const float* __restrict__ k_w,
                                    const float* __restrict__ inv_freq, const int* __restrict__ positions,
@@ -65,14 +70,16 @@ __global__ void qkv_prepare_kernel(T* __restrict__ q_out, T* __restrict__ k_cach
                                    int table_stride, int nh, int nkv, int d, int dv, int rot, int interleaved, int norm_mode,
                                    int page_size, int num_pages, float eps, int write_kv, int vec4, float rot_mag,
                                    const float* __restrict__ bias, float temp_coef, int temp_every, long long row_len,
-                                   long long v_off, int* err) {
+                                   long long v_off, const float* __restrict__ taps, int K, T* conv_state,
+                                   const int* __restrict__ q_start, const int* __restrict__ slots, int keep_state,
+                                   float value_eps, int* err) {
     extern __shared__ float sm[];
     __shared__ float red2[2][32];
     const int half = rot / 2;
     float* cs = sm;                 // [half]
     float* sn = sm + half;          // [half]
     const int nwarps = blockDim.x >> 5, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-    float* xs = sm + 2 * half + (size_t)warp * d;   // this warp's head
+    float* xs = sm + 2 * half + (size_t)warp * (dv > d && value_eps >= 0.f ? dv : d);   // this warp's head
     const int t = blockIdx.x;
     const int pos = positions[t];
     const int b = req_of_token[t];
@@ -96,6 +103,44 @@ __global__ void qkv_prepare_kernel(T* __restrict__ q_out, T* __restrict__ k_cach
         }
     }
     const T* row = qkv + (size_t)t * row_len;     // (a row may hold more behind its q, k and v)
+    const int C = (nh + nkv) * d + nkv * dv;      // channels of the convolution
+    int t0 = t, slot = -1;
+    if (CONV && b >= 0) {
+        t0 = q_start[b];
+        slot = slots[b];
+    }
+    // row j of the K that a token's convolution reads (nullptr: before the sequence's start)
+    auto conv_row = [&](int j) -> const T* {
+        const int src = t - (K - 1) + j;
+        if (src >= t0) return qkv + (size_t)src * row_len;
+        return slot >= 0 ? conv_state + ((size_t)slot * (K - 1) + (K - 1 + src - t0)) * C : nullptr;
+    };
+    // elements of the token's row (convolved) at a column of q, k or v
+    auto ld4 = [&](long long col, float (&v)[4]) {
+        if (!CONV) {
+            load4<T>(row + col, v);
+            return;
+        }
+        v[0] = v[1] = v[2] = v[3] = 0.f;
+        for (int j = 0; j < K; ++j) {
+            const T* p = conv_row(j);
+            if (p == nullptr) continue;
+            float u[4];
+            load4<T>(p + col, u);
+            const float4 w4 = *reinterpret_cast<const float4*>(taps + (size_t)j * C + col);
+            v[0] = fmaf(w4.x, u[0], v[0]); v[1] = fmaf(w4.y, u[1], v[1]);
+            v[2] = fmaf(w4.z, u[2], v[2]); v[3] = fmaf(w4.w, u[3], v[3]);
+        }
+    };
+    auto ld1 = [&](long long col) -> float {
+        if (!CONV) return to_f32<T>(row[col]);
+        float v = 0.f;
+        for (int j = 0; j < K; ++j) {
+            const T* p = conv_row(j);
+            if (p != nullptr) v = fmaf(taps[(size_t)j * C + col], to_f32<T>(p[col]), v);
+        }
+        return v;
+    };
     float inv_q = 1.f, inv_k = 1.f;
     if (norm_mode == 3) {     // one root mean square over the whole q projection, one over the whole k projection
         float sq = 0.f, sk = 0.f;
@@ -103,7 +148,7 @@ __global__ void qkv_prepare_kernel(T* __restrict__ q_out, T* __restrict__ k_cach
         if (vec4) {           // (d a multiple of 4: a group of four never straddles q and k)
             for (int i = threadIdx.x * 4; i < nqk; i += blockDim.x * 4) {
                 float v[4];
-                load4<T>(row + i, v);
+                ld4(i, v);
                 float s4 = 0.f;
 #pragma unroll
                 for (int k = 0; k < 4; ++k) {
@@ -114,7 +159,7 @@ __global__ void qkv_prepare_kernel(T* __restrict__ q_out, T* __restrict__ k_cach
             }
         } else {
             for (int i = threadIdx.x; i < nqk; i += blockDim.x) {
-                const float v = to_f32<T>(row[i]) + (bias ? bias[i] : 0.f);
+                const float v = ld1(i) + (bias ? bias[i] : 0.f);
                 if (i < nq) sq += v * v; else sk += v * v;
             }
         }
@@ -138,13 +183,46 @@ __global__ void qkv_prepare_kernel(T* __restrict__ q_out, T* __restrict__ k_cach
         if (h >= nh + nkv) {      // a value head: copy (plus its bias)
             if (kv_row < 0) continue;
             const int g = h - nh - nkv;
-            const T* x = row + v_off + (size_t)g * dv;
+            const long long xv = v_off + (long long)g * dv;
             const float* bv = bias ? bias + v_off + (size_t)g * dv : nullptr;
             T* dst = v_cache + (size_t)(kv_row + (long long)g * page_size) * dv;
+            if (value_eps >= 0.f) {     // of unit size: the head passes through shared memory
+                float ss = 0.f;
+                if (vec4) {
+                    for (int i = lane * 4; i < dv; i += 128) {
+                        float v[4];
+                        ld4(xv + i, v);
+#pragma unroll
+                        for (int k = 0; k < 4; ++k) {
+                            if (bv) v[k] += bv[i + k];
+                            ss = fmaf(v[k], v[k], ss);
+                        }
+                        *reinterpret_cast<float4*>(xs + i) = make_float4(v[0], v[1], v[2], v[3]);
+                    }
+                } else {
+                    for (int i = lane; i < dv; i += 32) {
+                        const float v = ld1(xv + i) + (bv ? bv[i] : 0.f);
+                        ss = fmaf(v, v, ss);
+                        xs[i] = v;
+                    }
+                }
+                const float inv = 1.f / sqrtf(warp_sum(ss) / (float)dv + value_eps);
+                if (vec4) {     // (a lane reads back what it wrote itself)
+                    for (int i = lane * 4; i < dv; i += 128) {
+                        const float4 f = *reinterpret_cast<const float4*>(xs + i);
+                        const float v[4] = {f.x * inv, f.y * inv, f.z * inv, f.w * inv};
+                        store4<T>(dst + i, v);
+                    }
+                } else {
+                    for (int i = lane; i < dv; i += 32) dst[i] = from_f32<T>(xs[i] * inv);
+                }
+                __syncwarp();
+                continue;
+            }
             if (vec4) {
                 for (int i = lane * 4; i < dv; i += 128) {
                     float v[4];
-                    load4<T>(x + i, v);
+                    ld4(xv + i, v);
                     if (bv) {
 #pragma unroll
                         for (int k = 0; k < 4; ++k) v[k] += bv[i + k];
@@ -152,15 +230,15 @@ __global__ void qkv_prepare_kernel(T* __restrict__ q_out, T* __restrict__ k_cach
                     store4<T>(dst + i, v);
                 }
             } else if (bv) {
-                for (int i = lane; i < dv; i += 32) dst[i] = from_f32<T>(to_f32<T>(x[i]) + bv[i]);
+                for (int i = lane; i < dv; i += 32) dst[i] = from_f32<T>(ld1(xv + i) + bv[i]);
             } else {
-                for (int i = lane; i < dv; i += 32) dst[i] = x[i];
+                for (int i = lane; i < dv; i += 32) dst[i] = from_f32<T>(ld1(xv + i));
             }
             continue;
         }
         const bool is_q = h < nh;
         if (!is_q && kv_row < 0) continue;
-        const T* x = row + (size_t)h * d;
+        const long long xc = (long long)h * d;
         const float* bh = bias ? bias + (size_t)h * d : nullptr;
         const float om = is_q ? q_mul : 1.f;
         T* dst = is_q ? q_out + ((size_t)t * nh + h) * d
@@ -173,7 +251,7 @@ __global__ void qkv_prepare_kernel(T* __restrict__ q_out, T* __restrict__ k_cach
             const float inv = norm_mode == 3 ? (is_q ? inv_q : inv_k) : 1.f;
             for (int i = lane * 4; i < d; i += 128) {
                 float v[4];
-                load4<T>(x + i, v);
+                ld4(xc + i, v);
                 if (bh) {
                     const float4 b4 = *reinterpret_cast<const float4*>(bh + i);
                     v[0] += b4.x; v[1] += b4.y; v[2] += b4.z; v[3] += b4.w;
@@ -202,7 +280,7 @@ __global__ void qkv_prepare_kernel(T* __restrict__ q_out, T* __restrict__ k_cach
             const float inv = is_q ? inv_q : inv_k;
             for (int i = lane * 4; i < d; i += 128) {
                 float v[4];
-                load4<T>(x + i, v);
+                ld4(xc + i, v);
 #pragma unroll
                 for (int k = 0; k < 4; ++k) {
                     if (bh) v[k] += bh[i + k];
@@ -212,7 +290,7 @@ __global__ void qkv_prepare_kernel(T* __restrict__ q_out, T* __restrict__ k_cach
         } else if (vec4) {
             for (int i = lane * 4; i < d; i += 128) {
                 float v[4];
-                load4<T>(x + i, v);
+                ld4(xc + i, v);
 #pragma unroll
                 for (int k = 0; k < 4; ++k) {
                     if (bh) v[k] += bh[i + k];
@@ -222,7 +300,7 @@ __global__ void qkv_prepare_kernel(T* __restrict__ q_out, T* __restrict__ k_cach
             }
         } else {
             for (int i = lane; i < d; i += 32) {
-                const float v = to_f32<T>(x[i]) + (bh ? bh[i] : 0.f);
+                const float v = ld1(xc + i) + (bh ? bh[i] : 0.f);
                 xs[i] = v;
                 ss += v * v;
             }
@@ -262,6 +340,14 @@ __global__ void qkv_prepare_kernel(T* __restrict__ q_out, T* __restrict__ k_cach
         }
         __syncwarp();
     }
+    if (CONV && keep_state && slot >= 0 && K > 1) {
+        __syncthreads();        // every warp has read the old rows
+        T* st = conv_state + (size_t)slot * (K - 1) * C;
+        for (int c = threadIdx.x; c < C; c += blockDim.x) {
+            for (int j = 0; j + 1 < K - 1; ++j) st[(size_t)j * C + c] = st[(size_t)(j + 1) * C + c];
+            st[(size_t)(K - 2) * C + c] = row[c];
+        }
+    }
 }
 
 XB_EXPORT int xb_qkv_prepare(int dtype, void* q_out, void* k_cache, void* v_cache, const void* qkv, const float* q_w,
@@ -269,33 +355,39 @@ XB_EXPORT int xb_qkv_prepare(int dtype, void* q_out, void* k_cache, void* v_cach
                              const int* block_table, int table_stride, int tokens, int nh, int nkv, int d, int dv, int rot,
                              int interleaved, int norm_mode, int page_size, int num_pages, float eps, int write_kv, float rot_mag,
                              const float* bias, float temp_coef, int temp_every, long long row_len, long long v_off,
-                             int* err, cudaStream_t stream) {
+                             const float* taps, int K, void* conv_state, const int* q_start, const int* slots, int keep_state,
+                             float value_eps, int* err, cudaStream_t stream) {
     if (tokens <= 0) return 0;
     if (v_off < 0) v_off = (long long)(nh + nkv) * d;
+    // the convolution takes q, k and v as they lie behind each other, and no bias
+    if (taps && (K < 1 || bias || v_off != (long long)(nh + nkv) * d || (K > 1 && !conv_state) || !q_start || !slots))
+        return (int)cudaErrorInvalidValue;
     // a warp per head at a time: as many warps as a token has heads, up to 16
     const int heads = nh + 2 * nkv;
     int threads = heads >= 16 ? 512 : (heads >= 8 ? 256 : 128);
-    size_t smem = ((size_t)rot + (size_t)(threads / 32) * d) * sizeof(float);
+    const int wide = value_eps >= 0.f && dv > d ? dv : d;
+    size_t smem = ((size_t)rot + (size_t)(threads / 32) * wide) * sizeof(float);
     while (smem > 48 * 1024 && threads > 32) {     // very wide heads: fewer warps, each still with room for its head
         threads /= 2;
-        smem = ((size_t)rot + (size_t)(threads / 32) * d) * sizeof(float);
+        smem = ((size_t)rot + (size_t)(threads / 32) * wide) * sizeof(float);
     }
     if (smem > 48 * 1024) return (int)cudaErrorInvalidValue;
     // four elements per access where every head starts on such a boundary, in the rows and in the pages
     const size_t esz = dtype == XB_F32 ? 4 : 2;
-    const int vec4 = (d % 4 == 0 && dv % 4 == 0 && row_len % 4 == 0 && v_off % 4 == 0 &&
-                      !(((uintptr_t)bias | (uintptr_t)q_w | (uintptr_t)k_w) & 15) &&
+    const int vec4 = (d % 4 == 0 && dv % 4 == 0 && row_len % 4 == 0 && v_off % 4 == 0 && (rot % 4 == 0 || value_eps < 0.f) &&
+                      !((uintptr_t)taps & 15) && !((uintptr_t)conv_state & (4 * esz - 1)) && !(((uintptr_t)bias | (uintptr_t)q_w | (uintptr_t)k_w) & 15) &&
                       !(((uintptr_t)qkv | (uintptr_t)q_out | (uintptr_t)k_cache | (uintptr_t)v_cache) & (4 * esz - 1))) ? 1 : 0;
-    if (dtype == XB_F32)
-        qkv_prepare_kernel<float><<<tokens, threads, smem, stream>>>(
-            (float*)q_out, (float*)k_cache, (float*)v_cache, (const float*)qkv, q_w, k_w, inv_freq, positions, req_of_token,
-            block_table, table_stride, nh, nkv, d, dv, rot, interleaved, norm_mode, page_size, num_pages, eps, write_kv, vec4, rot_mag,
-            bias, temp_coef, temp_every, row_len, v_off, err);
-    else
-        qkv_prepare_kernel<__nv_bfloat16><<<tokens, threads, smem, stream>>>(
-            (__nv_bfloat16*)q_out, (__nv_bfloat16*)k_cache, (__nv_bfloat16*)v_cache, (const __nv_bfloat16*)qkv, q_w, k_w,
-            inv_freq, positions, req_of_token, block_table, table_stride, nh, nkv, d, dv, rot, interleaved, norm_mode,
-            page_size, num_pages, eps, write_kv, vec4, rot_mag, bias, temp_coef, temp_every, row_len, v_off, err);
+#define XB_PREPARE(T, CONV)                                                                                               \
+    qkv_prepare_kernel<T, CONV><<<tokens, threads, smem, stream>>>(                                                      \
+        (T*)q_out, (T*)k_cache, (T*)v_cache, (const T*)qkv, q_w, k_w, inv_freq, positions, req_of_token, block_table,    \
+        table_stride, nh, nkv, d, dv, rot, interleaved, norm_mode, page_size, num_pages, eps, write_kv, vec4, rot_mag,   \
+        bias, temp_coef, temp_every, row_len, v_off, taps, K, (T*)conv_state, q_start, slots, keep_state, value_eps, err)
+    if (dtype == XB_F32) {
+        if (taps) XB_PREPARE(float, true); else XB_PREPARE(float, false);
+    } else {
+        if (taps) XB_PREPARE(__nv_bfloat16, true); else XB_PREPARE(__nv_bfloat16, false);
+    }
+#undef XB_PREPARE
     return xb_launch_status();
 }
 

@@ -292,20 +292,20 @@ class ModelRunner:
     # ---- caches --------------------------------------------------------------------------------------
     def _build_caches(self, num_blocks: Optional[int], kv_fraction: float) -> None:
         """Page pools and page tensors from what the mixers ask for.  Runs that own pages are
-        grouped by (window, page size): a group has one pool and one block table per request;
+        grouped by (window, first positions kept beside it, page size): a group has one pool and one block table per request;
         every run of a group holds its own page tensors, addressed by the group's page ids.
         ``num_blocks`` counts pages of the engine's ``block_size``; a group with another page size
         gets as many pages as hold the same number of tokens."""
         needs = self.model.cache_needs()
         runs = self.plan.runs
-        keys: List[Tuple[Optional[int], int]] = []
+        keys: List[Tuple[Optional[int], int, int]] = []
         run_group: Dict[int, int] = {}
         for pos, (run, need) in enumerate(zip(runs, needs)):
             if need is None or run.cache_from is not None:
                 continue
-            key = (need.window, int(need.page_size or self.block_size))
-            if key[1] <= 0:
-                raise StepError(f"layer run {pos} asks for a page size of {key[1]}")
+            key = (need.window, int(need.keep_first) if need.window else 0, int(need.page_size or self.block_size))
+            if key[2] <= 0:
+                raise StepError(f"layer run {pos} asks for a page size of {key[2]}")
             if key not in keys:
                 keys.append(key)
             run_group[pos] = keys.index(key)
@@ -322,7 +322,7 @@ class ModelRunner:
         self.num_blocks = int(num_blocks)
         self.kv_bytes_per_token = sum(token_bytes)
         tokens = self.num_blocks * self.block_size
-        groups = [CacheGroup(ps, max(tokens // ps, 1), w) for w, ps in keys]
+        groups = [CacheGroup(ps, max(tokens // ps, 1), w, first) for w, first, ps in keys]
         if not groups:
             # no mixer caches anything: one group of bookkeeping alone (no device memory) that never runs
             # out, so that requests still have lengths and slots

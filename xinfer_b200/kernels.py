@@ -310,14 +310,17 @@ def qk_norm_rope_write(q_out, k_cache, v_cache, qkv, q_w, k_w, cos_t, sin_t, pos
 
 
 def attention_plain(out, q, k_cache, v_cache, positions, req_of_token, block_table, table_stride, window, scale, err, *,
-                    sink=None, value_dim=None, softcap=None, slope_exponent=None, chunk=None):
+                    sink=None, value_dim=None, softcap=None, slope_exponent=None, chunk=None, keep_first: int = 0,
+                    out_scale: float = 1.0):
     """Attention of every token over its request's cached positions, one warp per (token, head), float32 scores,
-    softmax and value sums.  ``q`` is ``[T, heads, d]``, ``out`` ``[T, heads, dv]``.  The caches are
+    softmax and value sums.  ``q`` is ``[T, heads, d]``; ``out`` ``[T, heads, dv]``, whose tokens may lie further apart than
+    their heads * dv, receives ``out_scale`` times the result.  The caches are
     ``[page, kv_head, slot, d]`` and ``[page, kv_head, slot, dv]``; with ``value_dim`` the values are the first
     ``value_dim`` channels of the key rows themselves (``v_cache`` is then ignored).  ``sink`` (float32 per head):
     one more softmax entry of that score without a value.  ``softcap``: scores pass ``cap * tanh(s / cap)``;
     ``slope_exponent`` x: head h's score of a key ``dist`` positions back loses ``2^(-x (h + 1) / heads) * dist``
-    (after the cap); ``chunk``: a query sees the keys of its own chunk of that many positions, counted from the
+    (after the cap); ``keep_first``: that many positions at the sequence's start stay visible beside the window; ``chunk``:
+    a query sees the keys of its own chunk of that many positions, counted from the
     sequence's start, instead of a window."""
     T, nh, d = q.shape
     _need(q, "q", None, (T, nh, d))
@@ -332,9 +335,11 @@ def attention_plain(out, q, k_cache, v_cache, positions, req_of_token, block_tab
         dv = v_cache.shape[-1]
         _need(v_cache, "v_cache", q.dtype, (num_pages, nkv, page_size, dv))
         v_stride = dv
-    _need(out, "out", q.dtype, (T, nh, dv))
+    ldo = _token_stride(out, q.dtype, T, nh, dv)
     if sink is not None:
         _need(sink, "sink", torch.float32, (nh,))
+    if keep_first and not window:
+        raise KernelError("first positions are kept beside a window")
     if nh % nkv:
         raise KernelError(f"{nh} query heads do not divide into {nkv} key/value heads")
     if max(d, dv) > 1024:
@@ -342,8 +347,18 @@ def attention_plain(out, q, k_cache, v_cache, positions, req_of_token, block_tab
     _ok(kernels_lib().xb_attention_plain(
         dtype_code(q.dtype), out.data_ptr(), q.data_ptr(), nh * d, d, k_cache.data_ptr(), v_cache.data_ptr(), d, v_stride,
         _ptr(sink), positions.data_ptr(), req_of_token.data_ptr(), block_table.data_ptr(), int(table_stride), T, nh, nkv, d,
-        dv, page_size, num_pages, int(window or 0), float(scale), float(softcap or 0.0), float(slope_exponent or 0.0),
-        int(chunk or 0), err.data_ptr(), _stream()), "attention_plain")
+        dv, page_size, num_pages, int(window or 0), int(keep_first), float(scale), float(softcap or 0.0),
+        float(slope_exponent or 0.0), int(chunk or 0), ldo, float(out_scale), err.data_ptr(), _stream()), "attention_plain")
+
+
+def _token_stride(out, dtype, T: int, nh: int, dv: int) -> int:
+    """Elements between the tokens of an attention's output ``[T, heads, dv]``: heads and channels are dense, tokens
+    may lie further apart (the output is then a column range of wider rows)."""
+    if (not out.is_cuda or out.dtype != dtype or tuple(out.shape) != (T, nh, dv) or out.stride(2) != 1
+            or (nh > 1 and out.stride(1) != dv) or (T > 1 and out.stride(0) < nh * dv)):
+        raise KernelError(f"out: expected a {dtype} CUDA view of shape {(T, nh, dv)} with dense heads, got {tuple(out.shape)} "
+                          f"with strides {out.stride()}")
+    return int(out.stride(0)) if T > 1 else max(int(out.stride(0)), nh * dv)
 
 
 # activations of a gated feed-forward by code.  "swish_clamp" takes two parameters (limit, alpha): with
@@ -504,7 +519,7 @@ def attn_decode_plan_size(tokens: int, ctas: int, kv_heads: int) -> int:
 
 
 def attn_decode_plan(plan, positions, req_of_token, q_start, num_entries, window, dec_max, direct, tokens, min_keys,
-                     ctas, kv_heads, err) -> bool:
+                     ctas, kv_heads, err, keep_first: int = 0) -> bool:
     """Decide how the attention of the step's ``tokens`` small tokens is shared out (pieces of about
     1 / ``ctas`` of all keys, at least ``min_keys`` each) and write it to ``plan`` (int32,
     ``attn_decode_plan_size`` elements).  It must run before the step's first kernel when
@@ -513,7 +528,7 @@ def attn_decode_plan(plan, positions, req_of_token, q_start, num_entries, window
     if plan.numel() < attn_decode_plan_size(tokens, ctas, kv_heads):
         raise KernelError("the attention plan buffer is too small")
     rc = kernels_lib().xb_attn_decode_plan(plan.data_ptr(), positions.data_ptr(), req_of_token.data_ptr(), q_start.data_ptr(),
-                                           int(num_entries), int(window or 0), int(dec_max), int(bool(direct)), int(tokens),
+                                           int(num_entries), int(window or 0), int(keep_first), int(dec_max), int(bool(direct)), int(tokens),
                                            int(min_keys), int(ctas), int(kv_heads), err.data_ptr(), _stream())
     if rc == ERR_NOT_SUPPORTED:
         return False
@@ -523,7 +538,7 @@ def attn_decode_plan(plan, positions, req_of_token, q_start, num_entries, window
 
 def attn_decode_tc(out, part_o, part_ml, q, k_cache, v_cache, plan, block_table, table_stride, scale, dec_max,
                    splits_max, tokens, ctas, err, tickets=None, overlap: bool = True, softcap=None,
-                   slope_exponent=None) -> bool:
+                   slope_exponent=None, sink=None, keep_first: int = 0, out_scale: float = 1.0) -> bool:
     """The step's small tokens on tcgen05 tensor cores with TMA-fed pages, shared out as ``plan``
     says (``attn_decode_plan`` with the same tokens, ctas and kv heads).  A token and head in several
     pieces is merged through ``part_o`` / ``part_ml`` (float32, tokens*heads*splits_max*head_dim
@@ -532,14 +547,18 @@ def attn_decode_tc(out, part_o, part_ml, q, k_cache, v_cache, plan, block_table,
     start while the kernel before drains - only with a plan made before the step's first kernel.
     Returns False, having done nothing, for shapes the kernel does not take (a head size over
     128, a page size that is no power of two >= 8, more than 16 query heads per key/value head).
-    ``softcap`` / ``slope_exponent``: scores capped and biased by the distance as in ``attention_plain``."""
+    ``softcap`` / ``slope_exponent`` / ``sink`` / ``keep_first`` (as the plan was made) / ``out_scale`` and the layout of
+    ``out``: as in ``attention_plain``; values may have another size than keys (also a multiple of 16 up to 128)."""
     T, nh, d = q.shape
     _need(q, "q", torch.bfloat16, (T, nh, d))
-    _need(out, "out", torch.bfloat16, (T, nh, d))
     _need(k_cache, "k_cache", torch.bfloat16, (None, None, None, d))
-    _need(v_cache, "v_cache", torch.bfloat16, tuple(k_cache.shape))
-    _need(plan, "plan", torch.int32)
     num_pages, nkv, ps, _ = k_cache.shape
+    dv = v_cache.shape[-1]
+    _need(v_cache, "v_cache", torch.bfloat16, (num_pages, nkv, ps, dv))
+    ldo = _token_stride(out, torch.bfloat16, T, nh, dv)
+    if sink is not None:
+        _need(sink, "sink", torch.float32, (nh,))
+    _need(plan, "plan", torch.int32)
     if nh % nkv or d % 16:
         raise KernelError(f"tiled attention needs a head size in steps of 16 and heads divisible by key/value heads; "
                           f"got head size {d}, {nh}/{nkv} heads")
@@ -548,15 +567,15 @@ def attn_decode_tc(out, part_o, part_ml, q, k_cache, v_cache, plan, block_table,
     if splits_max > 1:
         _need(part_o, "part_o", torch.float32)
         _need(part_ml, "part_ml", torch.float32)
-        if part_o.numel() < tokens * nh * splits_max * d or part_ml.numel() < tokens * nh * splits_max * 2:
+        if part_o.numel() < tokens * nh * splits_max * dv or part_ml.numel() < tokens * nh * splits_max * 2:
             raise KernelError("attention scratch buffers are too small for the number of pieces per token")
         _need(tickets, "tickets", torch.int32)
         if tickets.numel() < tokens * nkv:
             raise KernelError("the attention ticket buffer is too small")
     rc = kernels_lib().xb_attn_decode_tc(
         out.data_ptr(), _ptr(part_o), _ptr(part_ml), q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), plan.data_ptr(),
-        block_table.data_ptr(), int(table_stride), T, nh, nkv, d, ps, num_pages, float(scale), float(softcap or 0.0),
-        float(slope_exponent or 0.0), int(dec_max),
+        block_table.data_ptr(), int(table_stride), T, nh, nkv, d, dv, ldo, ps, num_pages, int(keep_first), float(scale),
+        float(softcap or 0.0), float(slope_exponent or 0.0), _ptr(sink), float(out_scale), int(dec_max),
         int(splits_max), int(tokens), int(ctas), _ptr(tickets), int(bool(overlap)), err.data_ptr(), _stream())
     if rc == ERR_NOT_SUPPORTED:
         return False
@@ -649,7 +668,7 @@ PREFILL_TC_MAX_CTAS = 148   # one CTA of the tcgen05 prefill kernel per SM
 
 
 def attn_prefill_work(counts, starts, dec_max: int, window, heads: int, kv_heads: int, max_ctas: int = PREFILL_TC_MAX_CTAS,
-                      host_buffer=None):
+                      host_buffer=None, keep_first: int = 0):
     """The work list of ``attn_prefill_tc`` for a step whose entries bring ``counts`` tokens after
     ``starts`` cached ones (host arrays): the portions of more than ``dec_max`` tokens cut into items of
     128 queries of a pair of query heads (of single heads where pairs would be too few) and shared out among at most ``max_ctas`` CTAs, longest first
@@ -663,36 +682,40 @@ def attn_prefill_work(counts, starts, dec_max: int, window, heads: int, kv_heads
     host = host_buffer(cap) if host_buffer is not None else torch.empty(cap, dtype=torch.int32).pin_memory()
     ctas = ctypes.c_int(0)
     used = host_lib().xb_attn_prefill_work(len(counts), counts.ctypes.data, starts.ctypes.data, int(dec_max), int(window or 0),
-                                           int(heads), int(kv_heads), int(max_ctas), host.data_ptr(), cap, ctypes.byref(ctas))
+                                           int(keep_first), int(heads), int(kv_heads), int(max_ctas), host.data_ptr(), cap, ctypes.byref(ctas))
     if used < 0:
         raise KernelError("the prefill work list does not fit its buffer")
     return host[:max(int(used), 1)], int(ctas.value)
 
 
 def attn_prefill_tc(out, q, k_cache, v_cache, q_start, start_pos, block_table, table_stride, window, scale, work, ctas, err,
-                    softcap=None, slope_exponent=None) -> bool:
+                    softcap=None, slope_exponent=None, sink=None, keep_first: int = 0, out_scale: float = 1.0) -> bool:
     """Prefill attention on tcgen05 (TMA-fed; scores, probabilities and accumulators in tensor memory):
     128 queries of two query heads of a key/value head per work item; ``work`` (int32, on the device)
     and ``ctas`` come from ``attn_prefill_work`` for the same step, heads and window.  Returns False,
     having done nothing, for sizes it does not take (head size over 128, page size not a power of two
     from 8).  ``window`` is a mask code here and in the work list and the decode plan: w > 0 a sliding window, -c < 0
-    chunks of c positions counted from the sequence's start (``mask_code``).  ``softcap`` / ``slope_exponent``: scores
-    capped and biased by the distance as in ``attention_plain``."""
+    chunks of c positions counted from the sequence's start (``mask_code``).  ``softcap`` / ``slope_exponent`` / ``sink`` /
+    ``keep_first`` (as the work list was made) / ``out_scale`` and the layout of ``out``: as in ``attention_plain``; values
+    may have another size than keys (also a multiple of 16 up to 128)."""
     T, nh, d = q.shape
     _need(q, "q", torch.bfloat16, (T, nh, d))
-    _need(out, "out", torch.bfloat16, (T, nh, d))
     _need(k_cache, "k_cache", torch.bfloat16, (None, None, None, d))
-    _need(v_cache, "v_cache", torch.bfloat16, tuple(k_cache.shape))
-    _need(work, "work", torch.int32)
     num_pages, nkv, ps, _ = k_cache.shape
+    dv = v_cache.shape[-1]
+    _need(v_cache, "v_cache", torch.bfloat16, (num_pages, nkv, ps, dv))
+    ldo = _token_stride(out, torch.bfloat16, T, nh, dv)
+    if sink is not None:
+        _need(sink, "sink", torch.float32, (nh,))
+    _need(work, "work", torch.int32)
     if ctas <= 0:
         return True
     if work.numel() < ctas + 1:
         raise KernelError("the prefill work list is shorter than its table of CTAs")
     rc = kernels_lib().xb_attn_prefill_tc(
         out.data_ptr(), q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), q_start.data_ptr(), start_pos.data_ptr(),
-        block_table.data_ptr(), int(table_stride), T, nh, nkv, d, ps, num_pages, int(window or 0), float(scale),
-        float(softcap or 0.0), float(slope_exponent or 0.0), work.data_ptr(), int(ctas), err.data_ptr(), _stream())
+        block_table.data_ptr(), int(table_stride), T, nh, nkv, d, dv, ldo, ps, num_pages, int(window or 0), int(keep_first),
+        float(scale), float(softcap or 0.0), float(slope_exponent or 0.0), _ptr(sink), float(out_scale), work.data_ptr(), int(ctas), err.data_ptr(), _stream())
     if rc == ERR_NOT_SUPPORTED:
         return False
     _ok(rc, "attn_prefill_tc")
@@ -702,7 +725,7 @@ def attn_prefill_tc(out, q, k_cache, v_cache, q_start, start_pos, block_table, t
 # ---- attention with talking heads and a sink; gated recurrence; polynomial activation; table experts ----
 def qkv_prepare(q_out, k_cache, v_cache, qkv, q_w, k_w, inv_freq, positions, req_of_token, block_table, table_stride,
                 nh, nkv, d, dv, rot, interleaved, norm_mode, eps, write_kv, err, rot_magnitude: float = 1.0, bias=None,
-                q_temp=None, row_len=None, value_offset=None):
+                q_temp=None, row_len=None, value_offset=None, conv=None, value_eps=None):
     """Per q/k head of the packed ``qkv`` rows ``[heads*d | kv_heads*d | kv_heads*dv]``: norm over the head
     (``norm_mode`` 1: before the rotation, 2: after it, 0: none; weight ``q_w`` / ``k_w`` or none), rotation of
     the first ``rot`` channels by ``position * inv_freq`` (float32 angles formed in the kernel; ``inv_freq`` None:
@@ -711,7 +734,12 @@ def qkv_prepare(q_out, k_cache, v_cache, qkv, q_w, k_w, inv_freq, positions, req
     position p is multiplied, last of all, by ``1 + coef * ln(floor((p + 1) / every) + 1)``.  ``norm_mode`` 3: like 1
     with ONE root mean square over all q channels of a token (and one over all its k channels) and weights of
     ``heads * d`` (``kv_heads * d``) channels.  ``value_offset``: where in a row the values start (default: behind q
-    and k); the offset of k makes the keys as projected double as values, and rows then hold no values of their own."""
+    and k); the offset of k makes the keys as projected double as values, and rows then hold no values of their own.
+    ``conv`` = (taps ``[K, channels]`` float32, state ``[slots, K-1, channels]`` in the rows' type or None for one tap,
+    q_start, slots, single): every channel of q, k and v first passes a causal convolution over time whose K - 1 inputs
+    before a step's first token come from the state, which then receives the step's last K - 1 inputs - in the same launch
+    where every request brings one token (``single``).  ``value_eps``: value heads are divided by their root mean square
+    (this eps under the root) before they are cached."""
     T = qkv.shape[0]
     v_off = (nh + nkv) * d if value_offset is None else int(value_offset)
     need_len = max((nh + nkv) * d, v_off + nkv * dv)
@@ -735,12 +763,30 @@ def qkv_prepare(q_out, k_cache, v_cache, qkv, q_w, k_w, inv_freq, positions, req
             _need(w_, name, torch.float32, (n_ * d if norm_mode == 3 else d,))
     if inv_freq is not None:
         _need(inv_freq, "inv_freq", torch.float32, (rot // 2,))
-    _ok(kernels_lib().xb_qkv_prepare(
+    C = (nh + nkv) * d + nkv * dv
+    taps = conv_state = q_start = slots = None
+    K, single = 0, False
+    if conv is not None:
+        taps, conv_state, q_start, slots, single = conv
+        K = taps.shape[0]
+        if bias is not None or value_offset is not None or not (1 <= K <= CONV_MAX_TAPS):
+            raise KernelError(f"a convolution of q, k and v takes 1 to {CONV_MAX_TAPS} taps, no biases and values of their own")
+        _need(taps, "taps", torch.float32, (K, C))
+        if K > 1:
+            _need(conv_state, "conv_state", qkv.dtype, (None, K - 1, C))
+        _need(q_start, "q_start", torch.int32)
+        _need(slots, "slots", torch.int32)
+    lib = kernels_lib()
+    _ok(lib.xb_qkv_prepare(
         dtype_code(qkv.dtype), q_out.data_ptr(), _ptr(k_cache), _ptr(v_cache), qkv.data_ptr(), _ptr(q_w), _ptr(k_w),
         _ptr(inv_freq), positions.data_ptr(), req_of_token.data_ptr(), block_table.data_ptr(), int(table_stride), T, nh, nkv,
         d, dv, int(rot if inv_freq is not None else 0), int(bool(interleaved)), int(norm_mode), page_size, num_pages,
-        float(eps), int(bool(write_kv)), float(rot_magnitude), _ptr(bias), coef, every, row_len, v_off, err.data_ptr(),
-        _stream()), "qkv_prepare")
+        float(eps), int(bool(write_kv)), float(rot_magnitude), _ptr(bias), coef, every, row_len, v_off, _ptr(taps), K,
+        _ptr(conv_state) if K > 1 else None, _ptr(q_start), _ptr(slots), int(bool(single)),
+        -1.0 if value_eps is None else float(value_eps), err.data_ptr(), _stream()), "qkv_prepare")
+    if K > 1 and not single:
+        _ok(lib.xb_conv_state(dtype_code(qkv.dtype), conv_state.data_ptr(), qkv.data_ptr(), row_len, 0, q_start.data_ptr(),
+                              slots.data_ptr(), slots.numel(), C, K, _stream()), "conv_state")
 
 
 def attn_talking_tile(nh: int, d: int, dv: int, want: int) -> int:
@@ -1226,7 +1272,7 @@ def conv_silu(y, u, u_off, taps, bias, state, req_of_token, q_start, slots, num_
                          _ptr(state) if K > 1 else None, req_of_token.data_ptr(), q_start.data_ptr(), slots.data_ptr(), T, C, K,
                          _stream()), "conv_silu")
     if K > 1:
-        _ok(lib.xb_conv_state(state.data_ptr(), u.data_ptr(), u.shape[1], int(u_off), q_start.data_ptr(), slots.data_ptr(),
+        _ok(lib.xb_conv_state(F32, state.data_ptr(), u.data_ptr(), u.shape[1], int(u_off), q_start.data_ptr(), slots.data_ptr(),
                               int(num_entries), C, K, _stream()), "conv_state")
 
 
@@ -1337,22 +1383,94 @@ def stream_conv(out, x, taps, state, req_of_token, q_start, slots, num_entries, 
                            _stream()), "stream_conv")
     if K > 1 and not in_pass:
         s = x if sum_out is None else sum_out
-        _ok(lib.xb_conv_state(state.data_ptr(), s.data_ptr(), C, 0, q_start.data_ptr(), slots.data_ptr(), int(num_entries), C, K,
+        _ok(lib.xb_conv_state(F32, state.data_ptr(), s.data_ptr(), C, 0, q_start.data_ptr(), slots.data_ptr(), int(num_entries), C, K,
                               _stream()), "conv_state")
 
 
-def gated_head_norm(out, y, gate, g_off, weight, part, eps, gate_after: bool, silu_gate: bool = False):
+def gated_head_norm(out, y, gate, g_off, weight, part, eps, gate_after: bool, silu_gate: bool = False, *, div=None,
+                    out_scale: float = 1.0):
     """Per token and group of ``part`` channels of ``y`` (float32): with ``gate_after`` False,
     v = y * silu(gate), out = v / rms(v) * weight; with True, out = y / rms(y) * weight * sigmoid(gate), or silu(gate)
     for the last factor with ``silu_gate``.  ``gate`` is
-    the columns from ``g_off`` of float32 rows; ``weight`` repeats every ``weight.numel()`` channels."""
+    the columns from ``g_off`` of float32 rows; ``weight`` repeats every ``weight.numel()`` channels.  ``div`` (float32
+    ``[T, W / part]``): a group of y is divided by its number first of all.  ``out`` may be a column range of wider rows; it
+    receives ``out_scale`` times the result."""
     T, W = y.shape
     _need(y, "y", torch.float32, (T, W))
-    _need(out, "out", None, (T, W))
+    if tuple(out.shape) != (T, W) or out.stride(1) != 1 or not out.is_cuda:
+        raise KernelError("out must be a CUDA view [T, W] with unit column stride")
+    if div is not None:
+        _need(div, "div", torch.float32, (T, W // part))
     _need(gate, "gate", torch.float32, (T, None))
     _need(weight, "weight", torch.float32)
     if g_off < 0 or g_off + W > gate.shape[1] or W % part or W % weight.numel():
         raise KernelError("gate columns, group size or weight length do not fit the rows")
     _ok(kernels_lib().xb_gated_head_norm(dtype_code(out.dtype), out.data_ptr(), y.data_ptr(), gate.data_ptr(), gate.shape[1],
                                          int(g_off), weight.data_ptr(), weight.numel(), T, W, int(part), float(eps),
-                                         (2 if silu_gate else 1) if gate_after else 0, _stream()), "gated_head_norm")
+                                         (2 if silu_gate else 1) if gate_after else 0, _ptr(div), int(out.stride(0)),
+                                         float(out_scale), _stream()), "gated_head_norm")
+
+
+def matrix_memory(o, div, proj, gate_off, b_in, b_forget, cap: float, state, q_start, start_pos, slots, num_entries, heads, d,
+                  dv, scale: float, div_eps: float):
+    """A matrix memory with exponential gates per (request, head): with the log gates i = cap tanh((z_i + b_in) / cap) and
+    f = logsigmoid(cap tanh((z_f + b_forget) / cap)) and the running maximum m' = max(f + m, i),
+    S <- e^(f + m - m') S + e^(i - m') k v^T, n likewise with k alone; ``o`` ``[T, heads * dv]`` = scale S^T q and ``div``
+    ``[T, heads]`` = max(|scale n . q|, e^(-m')) + div_eps, both after the token's own write.  ``proj`` float32 rows
+    ``[q | k | v | ...]`` with z_i and z_f (heads each) from column ``gate_off``.  ``state``: "S" ``[slots, heads, d, dv]``,
+    "n" ``[slots, heads, d]`` and "m" ``[slots, heads, 2, 2]``, all zero at a request's start."""
+    T = proj.shape[0]
+    _need(proj, "proj", torch.float32, (T, None))
+    if proj.shape[1] < max(heads * (2 * d + dv), gate_off + 2 * heads) or gate_off < 0:
+        raise KernelError("q, k, v or the gates lie outside the projection's rows")
+    _need(o, "o", torch.float32, (T, heads * dv))
+    _need(div, "div", torch.float32, (T, heads))
+    _need(b_in, "b_in", torch.float32, (heads,))
+    _need(b_forget, "b_forget", torch.float32, (heads,))
+    _need(state["S"], "S", torch.float32, (None, heads, d, dv))
+    _need(state["n"], "n", torch.float32, (None, heads, d))
+    _need(state["m"], "m", torch.float32, (None, heads, 2, 2))
+    _need(start_pos, "start_pos", torch.int32)
+    _ok(kernels_lib().xb_matrix_memory(o.data_ptr(), div.data_ptr(), proj.data_ptr(), proj.shape[1], int(gate_off),
+                                       b_in.data_ptr(), b_forget.data_ptr(), float(cap), state["S"].data_ptr(),
+                                       state["n"].data_ptr(), state["m"].data_ptr(), q_start.data_ptr(), start_pos.data_ptr(),
+                                       slots.data_ptr(), int(num_entries), heads, d, dv, float(scale), float(div_eps),
+                                       _stream()), "matrix_memory")
+
+
+# ---- several residual streams ------------------------------------------------------------------------------------------
+def stream_mix(out, x, read, weight, eps, err, *, branch=None, mix=None, write=None, x_out=None, rows=None,
+               weight_offset: float = 0.0):
+    """One pass over a token's ``n`` float32 streams ``x`` ``[T, n, dim]`` (which may be one copy read n times: a stride of 0
+    between streams): ``X'[t] = sum_s mix[s, t] x[s] + write[t] * branch`` (no branch: X' = x), ``u = sum_t read[t] X'[t]``
+    (``read`` None: the plain sum).  ``x_out`` (``[T, n, dim]``; may be ``x``) receives X'; ``out`` (either type; None: only
+    X') receives ``u / rms(u) * (weight_offset + weight)``, or u itself where ``weight`` is None, gathered at ``rows``."""
+    src, n, dim = x.shape
+    if x.dtype != torch.float32 or not x.is_cuda or (dim > 1 and x.stride(2) != 1):
+        raise KernelError("x: expected float32 CUDA streams [T, n, dim] with dense channels")
+    nrows = out.shape[0] if out is not None else src
+    if out is not None:
+        _need(out, "out", None, (nrows, dim))
+    if branch is not None:
+        _need(branch, "branch", None, (src, dim))
+        _need(mix, "mix", torch.float32, (n, n))
+        _need(write, "write", torch.float32, (n,))
+    if read is not None:
+        _need(read, "read", torch.float32, (n,))
+    if weight is not None:
+        _need(weight, "weight", torch.float32, (dim,))
+    if x_out is not None:
+        _need(x_out, "x_out", torch.float32, (src, n, dim))
+        if x_out.data_ptr() == x.data_ptr() and not x.is_contiguous():
+            raise KernelError("streams that share one copy cannot be written in place")
+    if rows is not None:
+        _need(rows, "rows", torch.int32)
+        if rows.numel() < nrows or x_out is not None:
+            raise KernelError("gathered rows: a list of every output row, and no streams are stored")
+    elif nrows != src:
+        raise KernelError(f"out has {nrows} rows, x has {src} and no row list was given")
+    _ok(kernels_lib().xb_stream_mix(dtype_code(branch.dtype) if branch is not None else F32,
+                                    dtype_code(out.dtype) if out is not None else F32, _ptr(out), _ptr(x_out), x.data_ptr(),
+                                    x.stride(0), x.stride(1), _ptr(branch), _ptr(rows), _ptr(read), _ptr(mix), _ptr(write),
+                                    _ptr(weight), nrows, n, dim, src, float(eps), float(weight_offset), err.data_ptr(),
+                                    _stream()), "stream_mix")

@@ -2,7 +2,7 @@
 
 embedding (times the plan's ``embed_scale``, if it has one) -> the plan's layer runs in order (a run may add the
 embedding's output to the stream again: layers that are run several times in a row start every pass but the first so) ->
-final norm on the wanted rows -> output head -> the plan's logit scale and soft cap, if any.
+final norm on the wanted rows (of several residual streams: of their sum) -> output head -> the plan's logit scale and soft cap, if any.
 (The reference's forward for this architecture: src/models/qwen3.rs:311-374.)
 """
 from __future__ import annotations
@@ -15,7 +15,7 @@ import torch
 from .. import kernels, tracing
 from ..config.plan import ModelPlan
 from ..parts import Block, LayerCache, StepContext, build_part, part_class
-from ..parts.block import Addend, Stream, fused_norm
+from ..parts.block import Addend, Stream, fused_norm, stream_chain
 from ..parts.linear import linear
 from ..weights.loader import WeightSpec, WeightStore
 
@@ -91,6 +91,9 @@ class DecoderModel:
         for b in self.blocks:
             for t in b.gains.values():
                 count(t)
+            for ts in b.mixes.values():
+                for t in ts:
+                    count(t)
             for part in b.all_parts():
                 stack = [part]
                 while stack:
@@ -157,7 +160,8 @@ class DecoderModel:
             kernels.embedding(x, self.embed, ctx.token_ids, ctx.err, ctx.sampled, scale=self.plan.embed_scale)
         if trace:
             tracing.pop()
-        stream = Stream(x)
+        # several residual streams are n views of the embedding's output until the first sublayer has written to them
+        stream = Stream(x if self.plan.streams is None else x.unsqueeze(1).expand(T, self.plan.streams, H))
         x0 = None
         if any(run.add_input for run in self.plan.runs):
             # runs that add the embedding's output again: it is kept apart from the stream that the blocks change
@@ -176,7 +180,11 @@ class DecoderModel:
         if trace:
             tracing.push("head")
         y = ws.get("model.final", (R, H), self.dtype)
-        fused_norm(self.final_norm, y, stream.x, ctx, stream.settle(ctx, keep_last=True), rows=ctx.logit_rows)
+        if self.plan.streams is not None:       # the final norm reads the streams' plain sum
+            last = stream.settle(ctx, keep_last=True)
+            stream_chain(self.final_norm, y, stream.x, ctx, None, last, rows=ctx.logit_rows, store=False)
+        else:
+            fused_norm(self.final_norm, y, stream.x, ctx, stream.settle(ctx, keep_last=True), rows=ctx.logit_rows)
         linear(logits, y, self.head, ctx.err)
         if self.plan.logit_scale is not None or self.plan.logit_softcap is not None:
             kernels.logits_post(logits, self.plan.logit_scale, self.plan.logit_softcap)

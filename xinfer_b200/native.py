@@ -47,7 +47,7 @@ def _sig(lib, name, restype, argtypes):
 
 
 def _declare_host(lib):
-    _sig(lib, "xb_cm_create", c_void_p, [c_int, POINTER(c_int), POINTER(c_int), POINTER(c_int), c_int])
+    _sig(lib, "xb_cm_create", c_void_p, [c_int, POINTER(c_int), POINTER(c_int), POINTER(c_int), POINTER(c_int), c_int])
     _sig(lib, "xb_cm_destroy", None, [c_void_p])
     for name in ("xb_cm_open", "xb_cm_live_requests"):
         _sig(lib, name, c_int, [c_void_p])
@@ -58,7 +58,7 @@ def _declare_host(lib):
     _sig(lib, "xb_cm_copy_table", c_int, [c_void_p, c_int, c_int, _I32P, c_int])
     _sig(lib, "xb_cm_consistent", c_int, [c_void_p, c_char_p, c_int])
     _sig(lib, "xb_attn_prefill_work", c_longlong,
-         [c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_longlong, c_void_p])
+         [c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_longlong, c_void_p])
     _sig(lib, "xb_cm_log_freed", None, [c_void_p, c_int])
     _sig(lib, "xb_cm_drain_freed", c_int, [c_void_p, c_void_p, c_void_p, c_int])
     _sig(lib, "xb_assemble", c_longlong,
@@ -93,7 +93,8 @@ def _declare_kernels(lib):
     _sig(lib, "xb_rope_table", I, [P, P, P, I, I, P])
     _sig(lib, "xb_qk_norm_rope_write", I,
          [I, P, P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, I, F, I, P, P])
-    _sig(lib, "xb_attention_plain", I, [I, P, P, L, L, P, P, I, I, P, P, P, P, I, I, I, I, I, I, I, I, I, F, F, F, I, P, P])
+    _sig(lib, "xb_attention_plain", I,
+         [I, P, P, L, L, P, P, I, I, P, P, P, P, I, I, I, I, I, I, I, I, I, I, F, F, F, I, L, F, P, P])
     _sig(lib, "xb_swiglu", I, [I, P, P, I, I, I, F, F, P])
     _sig(lib, "xb_widen_bf16", I, [P, P, L, P])
     _sig(lib, "xb_sample", I, [P, P, P, P, I, I, I, I, P, P, P])
@@ -104,7 +105,7 @@ def _declare_kernels(lib):
     _sig(lib, "xb_qk_norm_rope_write_bf16", I,
          [P, P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, I, F, I, P, P])
     _sig(lib, "xb_swiglu_rows_bf16", I, [P, P, I, I, I, F, F, P])
-    _sig(lib, "xb_attn_prefill_tc", I, [P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, F, F, F, P, I, P, P])
+    _sig(lib, "xb_attn_prefill_tc", I, [P, P, P, P, P, P, P, I, I, I, I, I, I, L, I, I, I, I, F, F, F, P, F, P, I, P, P])
     _sig(lib, "xb_gemm_skinny_tc", I, [P, I, P, P, I, I, I, I, P, P])
     _sig(lib, "xb_gemm_skinny_swiglu", I, [P, P, P, I, I, I, I, P, P])
     _sig(lib, "xb_gemm_skinny_qkv", I,
@@ -113,11 +114,12 @@ def _declare_kernels(lib):
     _sig(lib, "xb_attn_decode_bf16", I,
          [P, P, P, P, P, P, P, P, P, I, P, I, I, I, I, I, I, I, F, I, I, I, I, I, P, P, P])
     _sig(lib, "xb_attn_decode_plan_size", c_longlong, [I, I, I])
-    _sig(lib, "xb_attn_decode_plan", I, [P, P, P, P, I, I, I, I, I, I, I, I, P, P])
+    _sig(lib, "xb_attn_decode_plan", I, [P, P, P, P, I, I, I, I, I, I, I, I, I, P, P])
     _sig(lib, "xb_embedding_f32", I, [I, P, P, P, P, I, I, I, I, F, P, P])
     _sig(lib, "xb_rmsnorm_f32", I, [I, I, P, P, P, P, P, P, I, I, I, F, F, P, P])
     _sig(lib, "xb_add_f32", I, [I, P, P, P, L, F, P])
-    _sig(lib, "xb_qkv_prepare", I, [I, P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, I, I, F, I, F, P, F, I, L, L, P, P])
+    _sig(lib, "xb_qkv_prepare", I, 
+         [I, P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, I, I, F, I, F, P, F, I, L, L, P, I, P, P, P, I, F, P, P])
     _sig(lib, "xb_rms_chain", I, [I, I, P, P, P, P, P, P, P, P, I, I, I, F, F, F, F, F, P, P])
     _sig(lib, "xb_dual_rms_sum", I, [I, P, P, P, P, P, I, I, F, F, F, F, P])
     _sig(lib, "xb_add_bias", I, [I, P, P, I, I, P])
@@ -126,13 +128,15 @@ def _declare_kernels(lib):
     _sig(lib, "xb_prev_store", I, [P, P, P, I, P, P, I, P])
     _sig(lib, "xb_token_gate", I, [I, P, P, P, I, I, P, P, I, P, I, I, I, P, P])
     _sig(lib, "xb_conv_silu", I, [I, P, P, L, I, P, P, P, P, P, P, I, I, I, P])
-    _sig(lib, "xb_conv_state", I, [P, P, L, I, P, P, I, I, I, P])
+    _sig(lib, "xb_conv_state", I, [I, P, P, L, I, P, P, I, I, I, P])
     _sig(lib, "xb_selective_scan", I, [P, P, I, P, L, I, P, P, P, P, P, P, I, I, I, I, I, P])
     _sig(lib, "xb_delta_rule", I, [P, P, I, P, L, I, P, L, P, P, P, P, P, I, I, I, I, I, F, P])
     _sig(lib, "xb_linear_scan", I, [P, P, L, P, P, P, P, I, I, I, I, F, P])
     _sig(lib, "xb_low_rank_decay", I, [P, P, L, P, P, I, I, I, F, P])
     _sig(lib, "xb_stream_conv", I, [I, P, P, P, P, P, P, P, P, P, P, I, I, I, F, F, F, I, P])
-    _sig(lib, "xb_gated_head_norm", I, [I, P, P, P, L, I, P, I, I, I, I, F, I, P])
+    _sig(lib, "xb_gated_head_norm", I, [I, P, P, P, L, I, P, I, I, I, I, F, I, P, L, F, P])
+    _sig(lib, "xb_matrix_memory", I, [P, P, P, L, I, P, P, F, P, P, P, P, P, P, I, I, I, I, F, F, P])
+    _sig(lib, "xb_stream_mix", I, [I, I, P, P, P, L, L, P, P, P, P, P, P, I, I, I, I, F, F, P, P])
     _sig(lib, "xb_dyt_norm", I, [I, I, I, P, P, P, P, P, P, P, P, F, P, P, P, I, I, I, P, P])
     _sig(lib, "xb_latent_prepare", I,
          [I, P, P, P, L, I, I, P, L, L, P, P, P, P, P, I, I, I, I, I, I, I, I, I, F, F, I, P, I, I, P, P, P])
@@ -153,4 +157,5 @@ def _declare_kernels(lib):
     _sig(lib, "xb_expert_gather", I, [I, P, P, P, P, I, I, I, I, P])
     _sig(lib, "xb_expert_combine", I, [I, P, P, P, I, I, I, P, P, P, P])
     _sig(lib, "xb_expert_router", I, [I, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, F, F, P])
-    _sig(lib, "xb_attn_decode_tc", I, [P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, F, F, F, I, I, I, I, P, I, P, P])
+    _sig(lib, "xb_attn_decode_tc", I,
+         [P, P, P, P, P, P, P, P, I, I, I, I, I, I, L, I, I, I, F, F, F, P, F, I, I, I, I, P, I, P, P])

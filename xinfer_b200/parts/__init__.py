@@ -4,7 +4,7 @@ from .base import (CacheTensor, FeedForward, LayerCache, Mixer, Norm, PagedCache
                    register_mixer, register_norm, register_position_encoding, unregister)
 from . import (norm, rope, attention, swiglu, talking_attention, min_gru, parallel, polynorm_mlp,  # noqa: F401
                table_experts, latent_attention, selective_state, gated_delta, token_side, routed_experts, gated_linear_attention,
-               input_conv)                                                           # (register the built-in kinds)
+               input_conv, matrix_memory)                                                           # (register the built-in kinds)
 from .block import Block
 
 __all__ = [

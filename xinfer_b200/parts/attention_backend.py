@@ -41,13 +41,16 @@ def set_tiled(flag: bool) -> None:
     _enabled = bool(flag)
 
 
-def decode_tc_takes(nh: int, nkv: int, d: int, page_size: int) -> bool:
-    return (DECODE_TC and d % 16 == 0 and 16 <= d <= 128 and nh // nkv <= 16 and page_size >= 8
-            and page_size & (page_size - 1) == 0)
+def _tc_sizes(d: int, dv) -> bool:
+    return all(n % 16 == 0 and 16 <= n <= 128 for n in (d, d if dv is None else dv))
 
 
-def prefill_tc_takes(d: int, page_size: int) -> bool:
-    return (d % 16 == 0 and 16 <= d <= 128 and page_size >= 8 and page_size & (page_size - 1) == 0
+def decode_tc_takes(nh: int, nkv: int, d: int, page_size: int, dv=None) -> bool:
+    return DECODE_TC and _tc_sizes(d, dv) and nh // nkv <= 16 and page_size >= 8 and page_size & (page_size - 1) == 0
+
+
+def prefill_tc_takes(d: int, page_size: int, dv=None) -> bool:
+    return (_tc_sizes(d, dv) and page_size >= 8 and page_size & (page_size - 1) == 0
             and kernels.attn_prefill_queries(d, PREFILL_WARPS) == 128)
 
 
@@ -132,84 +135,94 @@ class _PinnedRing:
 _work_ring = _PinnedRing()
 
 
-def _prefill_work(ctx, nh: int, nkv: int, window):
+def _prefill_work(ctx, nh: int, nkv: int, window, keep_first: int = 0):
     """The step's work list of the tcgen05 prefill kernel for this head layout and window, made once
     per step (natively, on the host) and sent before the step's first kernel; shared by all layers."""
-    key = ("attn_prefill_work", nh, nkv, window)
+    key = ("attn_prefill_work", nh, nkv, window, keep_first)
     made = ctx.scratch.get(key)
     if made is None:
         counts = np.diff(ctx.h_q_start[: ctx.real_entries + 1])
         host, ctas = kernels.attn_prefill_work(counts, ctx.h_start_pos[: ctx.real_entries], DEC_MAX, window, nh, nkv,
-                                               host_buffer=_work_ring.take)
+                                               host_buffer=_work_ring.take, keep_first=keep_first)
         made = (host.to(ctx.positions.device, non_blocking=True), ctas, host)
         _work_ring.sent()
         ctx.scratch[key] = made
     return made
 
 
-def _decode_plan(ctx, nh: int, nkv: int, d: int, page_size: int, window, stride: int, early: bool):
+def _decode_plan(ctx, nh: int, nkv: int, d: int, page_size: int, window, stride: int, early: bool, keep_first: int = 0,
+                 dv=None):
     """The step's plan of the tcgen05 decode kernel for this head layout and window: made once per
     step and shared by all layers.  ``early``: the call comes before the step's first kernel.
     Returns None when the kernel does not take the step, else (plan, ctas, splits_max, overlap)."""
-    key = ("attn_decode_plan", nh, nkv, d, page_size, window)
+    key = ("attn_decode_plan", nh, nkv, d, page_size, window, keep_first, dv or d)
     if key in ctx.scratch:
         return ctx.scratch[key]
     made = None
     plan = _plan(ctx, d)
     small = plan["small"]
-    if small and decode_tc_takes(nh, nkv, d, page_size) and small <= DECODE_TC_MAX_TOKENS:
+    if small and decode_tc_takes(nh, nkv, d, page_size, dv) and small <= DECODE_TC_MAX_TOKENS:
         bound = plan["bound"] if plan["bound"] is not None else stride * page_size
         ctas, splits_max = decode_tc_launch(bound, small, nkv)
-        buf = ctx.workspace.get(f"attn.plan.{nkv}.{window or 0}", (kernels.attn_decode_plan_size(small, ctas, nkv),), torch.int32)
+        name = f"attn.plan.{nkv}.{window or 0}" + (f".{keep_first}" if keep_first else "")
+        buf = ctx.workspace.get(name, (kernels.attn_decode_plan_size(small, ctas, nkv),), torch.int32)
         if kernels.attn_decode_plan(buf, ctx.positions, ctx.req_of_token, ctx.q_start, ctx.num_entries, window, DEC_MAX,
-                                    plan["direct"], small, DECODE_TC_MIN_KEYS, ctas, nkv, ctx.err):
+                                    plan["direct"], small, DECODE_TC_MIN_KEYS, ctas, nkv, ctx.err, keep_first):
             # a plan made in the middle of the step is read only after the kernel before has completed
             made = (buf, ctas, splits_max, bool(early))
     ctx.scratch[key] = made
     return made
 
 
-def prepare_step(ctx, dtype, nh: int, nkv: int, d: int, page_size: int, window, stride: int) -> None:
+def prepare_step(ctx, dtype, nh: int, nkv: int, d: int, page_size: int, window, stride: int, *, keep_first: int = 0,
+                 dv=None) -> None:
     """Called before the step's first kernel for every attention layer (``stride``: the width of
     its block table): plans the decode kernel."""
     if _enabled and kernels.attn_tiled_supported(dtype, d):
-        _decode_plan(ctx, nh, nkv, d, page_size, window, stride, early=True)
-        if _plan(ctx, d)["tiles"] and PREFILL_TC and prefill_tc_takes(d, page_size):
-            _prefill_work(ctx, nh, nkv, window)
+        _decode_plan(ctx, nh, nkv, d, page_size, window, stride, early=True, keep_first=keep_first, dv=dv)
+        if _plan(ctx, d)["tiles"] and PREFILL_TC and prefill_tc_takes(d, page_size, dv):
+            _prefill_work(ctx, nh, nkv, window, keep_first)
 
 
-def takes_changed_scores(dtype, nh: int, nkv: int, d: int, page_size: int) -> bool:
-    """Capped scores, a distance bias and a chunked mask are built into the tcgen05 kernels only: whether they
-    take both the long portions and the single tokens of this layout."""
+def takes_changed_scores(dtype, nh: int, nkv: int, d: int, page_size: int, dv=None) -> bool:
+    """Capped scores, a distance bias, a chunked mask, a sink, kept first positions, values of another size than keys
+    and outputs that are scaled or lie apart are built into the tcgen05 kernels only: whether they take both the long
+    portions and the single tokens of this layout."""
     return (_enabled and PREFILL_TC and DECODE_TC and kernels.attn_tiled_supported(dtype, d)
-            and prefill_tc_takes(d, page_size) and decode_tc_takes(nh, nkv, d, page_size))
+            and prefill_tc_takes(d, page_size, dv) and decode_tc_takes(nh, nkv, d, page_size, dv))
 
 
-def attend(out, q, cache, ctx, table, stride, window, scale, *, softcap=None, slope_exponent=None, chunk=None) -> None:
+def attend(out, q, cache, ctx, table, stride, window, scale, *, softcap=None, slope_exponent=None, chunk=None, sink=None,
+           keep_first: int = 0, out_scale: float = 1.0) -> None:
     """``window``: a sliding window, or the mask code of ``kernels.mask_code`` (as ``prepare_step`` got it).
     ``softcap`` / ``slope_exponent`` / ``chunk``: scores capped and biased by the distance, keys of the query's
-    own chunk only; these run on the tcgen05 kernels or, where those do not take the step, on the plain one."""
+    own chunk only; ``sink``: one more softmax entry per head, of that score, without a value; ``keep_first``: the
+    sequence's first positions stay visible beside the window; ``out`` ``[T, heads, dv]`` receives ``out_scale`` times the
+    result and its tokens may lie apart.  These run on the tcgen05 kernels or, where those do not take the step, on the
+    plain one."""
     T, nh, d = q.shape
     k_pages, v_pages = cache["k"], cache["v"]
-    changed = softcap is not None or slope_exponent is not None or chunk is not None
+    dv = v_pages.shape[-1]
+    changed = (softcap is not None or slope_exponent is not None or chunk is not None or sink is not None or keep_first > 0
+               or out_scale != 1.0 or dv != d or not out.is_contiguous())
     if chunk is not None:
         window = kernels.mask_code(window, chunk)
 
     def plain():
         kernels.attention_plain(out, q, k_pages, v_pages, ctx.positions, ctx.req_of_token, table, stride,
-                                window if chunk is None else None, scale, ctx.err, softcap=softcap,
-                                slope_exponent=slope_exponent, chunk=chunk)
+                                window if chunk is None else None, scale, ctx.err, sink=sink, softcap=softcap,
+                                slope_exponent=slope_exponent, chunk=chunk, keep_first=keep_first, out_scale=out_scale)
 
     if not (_enabled and kernels.attn_tiled_supported(q.dtype, d)) or (
-            changed and not takes_changed_scores(q.dtype, nh, k_pages.shape[1], d, cache.page_size)):
+            changed and not takes_changed_scores(q.dtype, nh, k_pages.shape[1], d, cache.page_size, dv)):
         plain()
         return
     plan = _plan(ctx, d)
     took = False
-    if plan["tiles"] and PREFILL_TC and prefill_tc_takes(d, cache.page_size):
-        work, ctas, _ = _prefill_work(ctx, nh, k_pages.shape[1], window)
+    if plan["tiles"] and PREFILL_TC and prefill_tc_takes(d, cache.page_size, dv):
+        work, ctas, _ = _prefill_work(ctx, nh, k_pages.shape[1], window, keep_first)
         took = kernels.attn_prefill_tc(out, q, k_pages, v_pages, ctx.q_start, ctx.start_pos, table, stride, window, scale,
-                                       work, ctas, ctx.err, softcap, slope_exponent)
+                                       work, ctas, ctx.err, softcap, slope_exponent, sink, keep_first, out_scale)
     if plan["tiles"] and not took and changed:
         plain()         # (every token of the step, the small ones included)
         return
@@ -225,7 +238,7 @@ def attend(out, q, cache, ctx, table, stride, window, scale, *, softcap=None, sl
         def scratch(splits):
             nonlocal part_o, part_ml, tickets
             if splits > 1:
-                part_o = ctx.workspace.get("attn.part_o", (small * nh * splits * d,), torch.float32)
+                part_o = ctx.workspace.get("attn.part_o", (small * nh * splits * max(d, dv),), torch.float32)
                 part_ml = ctx.workspace.get("attn.part_ml", (small * nh * splits * 2,), torch.float32)
                 # zero-filled when made, left zero by the kernels; sized for either kernel
                 tickets = ctx.workspace.get("attn.tickets", (small * nkv * ((nh // nkv + 15) // 16),), torch.int32)
@@ -233,12 +246,13 @@ def attend(out, q, cache, ctx, table, stride, window, scale, *, softcap=None, sl
         step = (q, k_pages, v_pages, ctx.positions, ctx.req_of_token, ctx.q_start, ctx.num_entries, table, stride,
                 window, scale, DEC_MAX, plan["direct"])
         took = False
-        planned = _decode_plan(ctx, nh, nkv, d, cache.page_size, window, stride, early=False)
+        planned = _decode_plan(ctx, nh, nkv, d, cache.page_size, window, stride, early=False, keep_first=keep_first, dv=dv)
         if planned is not None:
             buf, ctas, splits_max, overlap = planned
             scratch(splits_max)
             took = kernels.attn_decode_tc(out, part_o, part_ml, q, k_pages, v_pages, buf, table, stride, scale, DEC_MAX,
-                                          splits_max, small, ctas, ctx.err, tickets, overlap, softcap, slope_exponent)
+                                          splits_max, small, ctas, ctx.err, tickets, overlap, softcap, slope_exponent, sink,
+                                          keep_first, out_scale)
         if not took and changed:
             if plan["tiles"]:
                 raise kernels.KernelError("a step of long portions and more single tokens than a plan takes, with changed scores")

@@ -128,12 +128,13 @@ class CacheTensor:
 class PagedCacheNeed:
     """What a mixer wants from the paged cache: named tensors per token (keys and values for
     attention, one latent vector for a mixer that caches that, ...), how long tokens are kept
-    (``window`` None keeps all) and, if it matters to its kernels, the page size (None: the
-    engine's).  Mixers with the same window and page size share a page pool and block tables."""
+    (``window`` None keeps all; ``keep_first`` positions at a sequence's start stay beside a window) and, if it matters to its kernels, the page size (None: the
+    engine's).  Mixers with the same retention and page size share a page pool and block tables."""
 
     tensors: Tuple[Tuple[str, CacheTensor], ...]
     window: Optional[int] = None
     page_size: Optional[int] = None
+    keep_first: int = 0
 
     @staticmethod
     def keys_and_values(kv_heads: int, head_dim: int, window: Optional[int] = None,

@@ -12,6 +12,8 @@ boundary: the last addition of a block waits in the ``Stream`` that the next blo
 decoder's final norm) receives.  A mixer whose first kernel can form the sum (``Mixer.takes_stream``) does
 so where it reads the stream itself.  Where a mixer or a feed-forward runs next, an addition kernel
 runs first (for every waiting addition: the part may reuse the buffer an addend lives in).
+Where the residual stream is several streams (``BlockOp.mix``), one kernel writes a sublayer's result to all of them,
+forms the weighted sum the next sublayer reads and norms it (``kernels.stream_mix``).
 The pre-norm block therefore launches exactly the kernels a hand-written one would.
 """
 from __future__ import annotations
@@ -42,11 +44,12 @@ def _width_of(spec: BlockSpec) -> int:
 class Addend:
     """A value that waits to be added into another: ``scale * gain * norm(t)``, where ``norm`` (a norm part, or None)
     has not been carried out yet - the kernel that forms the sum may do it, if its kind offers that - and ``gain`` is
-    a learned vector over the channels (or None)."""
+    a learned vector over the channels (or None).  ``mix``: the target is several streams; (M, w) of ``StreamMixSpec``."""
 
-    __slots__ = ("t", "scale", "norm", "gain")
+    __slots__ = ("t", "scale", "norm", "gain", "mix")
 
-    def __init__(self, t: torch.Tensor, scale: float = 1.0, norm=None, gain=None):
+    def __init__(self, t: torch.Tensor, scale: float = 1.0, norm=None, gain=None, mix=None):
+        self.mix = mix
         self.t = t
         self.scale = scale
         self.norm = norm
@@ -102,8 +105,35 @@ def fused_norm(part, out, src, ctx, last: Optional[Addend], rows=None):
     return part.forward(out, src, ctx, branch=last.t, sum_out=src, **kw)
 
 
+def stream_chain(part, out, x, ctx, read, last: Optional[Addend], rows=None, store: bool = True):
+    """``out = part(sum_s read[s] X[s])`` over several residual streams ``x`` ``[T, n, width]`` after the waiting addition
+    ``last``, in one kernel (``part`` None: only the addition); ``read`` None: the plain sum.  Returns the streams after the
+    addition, which lie in a buffer of their own where the old ones were n views of one copy (``store`` False: nobody
+    reads them again)."""
+    kw = {}
+    streams = x
+    if last is not None:
+        if store:
+            streams = x if x.is_contiguous() else ctx.workspace.get("model.streams", tuple(x.shape), torch.float32)
+            kw["x_out"] = streams
+        kw.update(branch=last.plain(ctx), mix=last.mix[0], write=last.mix[1])
+    if part is None:
+        if last is not None:
+            kernels.stream_mix(None, x, None, None, 0.0, ctx.err, **kw)
+    elif isinstance(part, RMSNorm):
+        ident = part.weight is None
+        kernels.stream_mix(out, x, read, part.weight, 0.0 if ident else part.spec.eps, ctx.err, rows=rows,
+                           weight_offset=0.0 if ident else part.spec.weight_offset, **kw)
+    else:       # a norm of another kind: the sum is formed first
+        u = ctx.workspace.get("block.streams_sum", tuple(out.shape), torch.float32)
+        kernels.stream_mix(u, x, read, None, 0.0, ctx.err, rows=rows, **kw)
+        part.forward(out, u, ctx)
+    return streams
+
+
 class Stream:
-    """The residual stream between blocks: its tensor and the branches still to be added to it."""
+    """The residual stream between blocks: its tensor (of several streams: ``[T, n, width]``) and the branches still to be
+    added to it."""
 
     __slots__ = ("x", "pending")
 
@@ -116,7 +146,10 @@ class Stream:
         norm kernel to fuse."""
         last = self.pending.pop() if (keep_last and self.pending) else None
         for b in self.pending:
-            _add_into(self.x, b, ctx)
+            if b.mix is not None:
+                self.x = stream_chain(None, None, self.x, ctx, None, b)
+            else:
+                _add_into(self.x, b, ctx)
         self.pending = []
         return last
 
@@ -137,6 +170,7 @@ class Block:
         self.mixer = mixers[0] if mixers else None
         self.device = device
         self.gains: Dict[str, torch.Tensor] = {}      # learned vectors of the additions, by tensor name after the prefix
+        self.mixes: Dict[Tuple[str, str, str], Tuple[torch.Tensor, ...]] = {}     # (r, M, w) of several residual streams
 
     @staticmethod
     def weight_specs(spec: BlockSpec) -> List[WeightSpec]:
@@ -149,6 +183,8 @@ class Block:
             out += part_class(_FAMILY[o.op], o.spec.kind).weight_specs(o.spec, spec.prefix + o.name)
         for name in sorted({o.gain for o in spec.program if o.op == "add" and o.gain is not None}):
             out.append(WeightSpec(spec.prefix + name, (_width_of(spec),), "norm"))
+        for names, n in sorted({(o.mix.names, o.mix.count) for o in spec.program if o.mix is not None}):
+            out += [WeightSpec(spec.prefix + name, shape, "unit") for name, shape in zip(names, ((n,), (n, n), (n,)))]
         return out
 
     def all_parts(self) -> List[Part]:
@@ -160,6 +196,9 @@ class Block:
         for o in self.spec.program:
             if o.op == "add" and o.gain is not None and o.gain not in self.gains:
                 self.gains[o.gain] = store.get(self.spec.prefix + o.gain, self.device, torch.float32).float().contiguous()
+            if o.mix is not None and o.mix.names not in self.mixes:
+                self.mixes[o.mix.names] = tuple(store.get(self.spec.prefix + n, self.device, torch.float32).float().contiguous()
+                                                for n in o.mix.names)
 
     def forward(self, stream: Stream, ctx: StepContext, cache: Optional[LayerCache], state, writes_cache: bool) -> Stream:
         """Runs the program on the residual stream; returns the stream with the additions that
@@ -176,7 +215,10 @@ class Block:
                 part = lazy.pop(name)
                 part.forward(t, t, ctx)
             for b in waiting.pop(name, ()):
-                _add_into(t, b, ctx)
+                if b.mix is not None:
+                    vals[name] = t = stream_chain(None, None, t, ctx, None, b)
+                else:
+                    _add_into(t, b, ctx)
             return t
 
         def settle_all() -> None:
@@ -188,6 +230,10 @@ class Block:
         for idx, o in enumerate(program):
             if o.op == "add":
                 gain = self.gains[o.gain] if o.gain is not None else None
+                if o.mix is not None:
+                    _, m, w = self.mixes[o.mix.names]
+                    waiting.setdefault(o.dst, []).append(Addend(read(o.src), mix=(m, w)))
+                    continue
                 if o.src in lazy and not waiting.get(o.src):
                     waiting.setdefault(o.dst, []).append(Addend(vals[o.src], o.scale, lazy.pop(o.src), gain))
                 else:
@@ -207,6 +253,21 @@ class Block:
                 if o.src in lazy:
                     read(o.src)
                 adds = waiting.pop(o.src, [])
+                if o.mix is not None:
+                    for b in adds[:-1]:
+                        src = stream_chain(None, None, src, ctx, None, b)
+                    out = ws.get("block." + o.dst, (src.shape[0], src.shape[2]), self.dtype)
+                    if adds and adds[-1].t.data_ptr() == out.data_ptr():
+                        out = ws.get("block." + o.dst + "'", tuple(out.shape), self.dtype)
+                    if tracing.ENABLED:
+                        tracing.push("norm")
+                    vals["x"] = stream_chain(part, out, src, ctx, self.mixes[o.mix.names][0], adds[-1] if adds else None)
+                    if tracing.ENABLED:
+                        tracing.pop()
+                    vals[o.dst] = out
+                    waiting.pop(o.dst, None)
+                    lazy.pop(o.dst, None)
+                    continue
                 for b in adds[:-1]:
                     _add_into(src, b, ctx)
                 last = adds[-1] if adds else None

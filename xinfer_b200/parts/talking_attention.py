@@ -12,7 +12,10 @@ Options of the spec beyond that: biases on q, k, v (and the output projection); 
 over the whole q (k) projection instead of one per head; a cap on the scores, ``cap * tanh(s / cap)``; a bias on
 the distance after the cap, ``- 2^(-x (h + 1) / heads) * (i - j)``; a chunked mask (a query sees the earlier keys
 of its own chunk of positions, counted from the sequence's start); a sigmoid gate on the heads' outputs, one number
-per channel or per head.
+per channel or per head; a window beside which the sequence's first positions stay visible (``keep_first``); a learned
+score per head as one more softmax entry without a value (``sink_name``); a causal convolution over time directly behind
+the projections (``conv``, its last inputs per-request state in the engine's type) and values divided by their root mean
+square before they are cached (``value_norm_eps``), both in the kernel that prepares q, k and v.
 
 Causal, optionally within a window; query head h reads key/value head h // (heads / kv_heads).  With a
 sink the weights of a row sum to less than one: a query may attend to nothing.  Keys after rotation and
@@ -56,6 +59,7 @@ class TalkingAttention(Mixer):
             raise ValueError("this attention needs a rotary position encoding that offers its frequencies")
         self.names = tuple(spec.names) if spec.names else _DEFAULT_NAMES
         self.w_qkv = self.w_o = self.talk = self.q_norm = self.k_norm = self.bias = self.b_o = None
+        self.sink_scores = self.taps = None
         if spec.value_from_key and spec.value_dim != spec.head_dim:
             raise ValueError(f"keys of {spec.head_dim} channels cannot double as values of {spec.value_dim}")
         if spec.chunk is not None and spec.window is not None:
@@ -63,6 +67,12 @@ class TalkingAttention(Mixer):
         if (spec.score_softcap is not None or spec.distance_slope_exponent is not None or spec.chunk is not None) and (
                 spec.talking_heads or spec.sink):
             raise ValueError("a score cap, a distance bias and a chunked mask are not built for talking heads or a sink")
+        if spec.keep_first and spec.window is None:
+            raise ValueError("first positions are kept beside a window")
+        if (spec.sink_name or spec.keep_first) and (spec.talking_heads or spec.sink):
+            raise ValueError("a learned sink and kept first positions are not built for talking heads or a silent sink")
+        if spec.conv is not None and (spec.bias_suffix or spec.value_from_key or not (1 <= spec.conv <= kernels.CONV_MAX_TAPS)):
+            raise ValueError(f"a convolution of q, k and v takes 1 to {kernels.CONV_MAX_TAPS} taps, no biases and values of their own")
 
     @classmethod
     def weight_specs(cls, spec: AttentionSpec, prefix: str) -> List[WeightSpec]:
@@ -88,6 +98,11 @@ class TalkingAttention(Mixer):
                 out.append(WeightSpec(prefix + n[2] + spec.bias_suffix, (spec.num_kv_heads * dv,), "around_zero"))
             if spec.out_bias:
                 out.append(WeightSpec(prefix + n[3] + spec.bias_suffix, (spec.hidden,), "around_zero"))
+        if spec.conv is not None:
+            rows = (spec.num_heads * d, spec.num_kv_heads * d, spec.num_kv_heads * dv)
+            out += [WeightSpec(prefix + n[i] + spec.conv_suffix, (rows[i], spec.conv), "unit") for i in range(3)]
+        if spec.sink_name:
+            out.append(WeightSpec(prefix + spec.sink_name, (spec.num_heads,), "unit"))
         if spec.gate_name:
             out.append(WeightSpec(prefix + spec.gate_name, (spec.num_heads * (1 if spec.gate_per_head else dv), spec.hidden)))
         return out
@@ -106,6 +121,11 @@ class TalkingAttention(Mixer):
             if s.out_bias:
                 self.b_o = store.get(p + n[3] + s.bias_suffix, self.device, torch.float32).float().contiguous()
         self.w_o = store.get(p + n[3], self.device, self.dtype, operand=True)
+        if s.conv is not None:      # [taps, channels of q, k and v]: neighbouring channels lie side by side
+            self.taps = torch.cat([store.get(p + n[i] + s.conv_suffix, self.device, torch.float32).float()
+                                   for i in range(3)]).t().contiguous()
+        if s.sink_name:
+            self.sink_scores = store.get(p + s.sink_name, self.device, torch.float32).float().contiguous()
         if s.talking_heads:
             self.talk = store.get(p + n[4], self.device, torch.float32).float().contiguous()
         if s.qk_norm and s.qk_norm_weight:
@@ -116,14 +136,22 @@ class TalkingAttention(Mixer):
     def cache_need(self) -> PagedCacheNeed:
         s = self.spec
         return PagedCacheNeed((("k", CacheTensor((s.num_kv_heads, s.head_dim), None, 1)),
-                               ("v", CacheTensor((s.num_kv_heads, s.value_dim), None, 1))), s.window)
+                               ("v", CacheTensor((s.num_kv_heads, s.value_dim), None, 1))), s.window, keep_first=s.keep_first)
+
+    def state_need(self):
+        s = self.spec
+        if s.conv is None or s.conv == 1:
+            return None
+        channels = (s.num_heads + s.num_kv_heads) * s.head_dim + s.num_kv_heads * s.value_dim
+        return {"conv": ((s.conv - 1, channels), self.dtype)}
 
     def _plain_softmax(self) -> bool:
-        """No mix across heads, no sink, key and value heads of one size in bfloat16: the attention itself is the
-        ordinary grouped-query one, and the engine's tcgen05 kernels (work lists, decode plans) take it."""
+        """No mix across heads, no silent sink, in bfloat16: the attention itself is the ordinary grouped-query one
+        (perhaps with a learned sink), and the engine's tcgen05 kernels (work lists, decode plans) may take it."""
         s = self.spec
-        return (USE_ATTENTION_BACKEND and not s.talking_heads and not s.sink and s.value_dim == s.head_dim
-                and self.dtype == torch.bfloat16 and kernels.attn_tiled_supported(self.dtype, s.head_dim))
+        return (USE_ATTENTION_BACKEND and not s.talking_heads and not s.sink and self.dtype == torch.bfloat16
+                and kernels.attn_tiled_supported(self.dtype, s.head_dim)
+                and (s.value_dim == s.head_dim or (s.value_dim % 16 == 0 and max(s.value_dim, s.head_dim) <= 128)))
 
     def _changed_scores(self) -> bool:
         """A cap, a distance bias or a chunked mask: what the ordinary attention kernels do not know."""
@@ -135,7 +163,8 @@ class TalkingAttention(Mixer):
             from . import attention_backend
             s = self.spec
             attention_backend.prepare_step(ctx, self.dtype, s.num_heads, s.num_kv_heads, s.head_dim, cache.page_size,
-                                           kernels.mask_code(s.window, s.chunk), ctx.strides[cache.group])
+                                           kernels.mask_code(s.window, s.chunk), ctx.strides[cache.group],
+                                           keep_first=s.keep_first, dv=s.value_dim)
 
     # ---- the two halves ---------------------------------------------------------------------------
     def inner_width(self) -> int:
@@ -166,7 +195,10 @@ class TalkingAttention(Mixer):
                             table, stride, nh, nkv, d, dv, rope.rotary_dim if rope is not None else 0,
                             rope is not None and rope.layout == "interleaved", norm_mode, s.qk_norm_eps, writes_cache,
                             ctx.err, rot_magnitude=rope.magnitude if rope is not None else 1.0, bias=self.bias,
-                            q_temp=s.q_temp, row_len=qkv.shape[1], value_offset=nh * d if s.value_from_key else None)
+                            q_temp=s.q_temp, row_len=qkv.shape[1], value_offset=nh * d if s.value_from_key else None,
+                            conv=(self.taps, (state or {}).get("conv"), ctx.q_start, ctx.slots,
+                                  ctx.all_single or ctx.fixed_shapes) if s.conv is not None else None,
+                            value_eps=s.value_norm_eps)
         self._attend(q, ctx, cache, table, stride, out, out_scale)
         if s.gate_name:
             kernels.gate_sigmoid(out, out.view(T, nh, dv).transpose(0, 1), qkv[:, nqkv:])
@@ -176,10 +208,21 @@ class TalkingAttention(Mixer):
         T = q.shape[0]
         nh, nkv, d, dv = s.num_heads, s.num_kv_heads, s.head_dim, s.value_dim
         ws = ctx.workspace
-        if self._plain_softmax() and out_scale == 1.0 and out.is_contiguous():
+        heads_out = out.unflatten(1, (nh, dv))
+        special = s.sink_name is not None or s.keep_first > 0       # what the kernels for talking heads do not know
+        if self._plain_softmax():
             from . import attention_backend
-            attention_backend.attend(out.view(T, nh, dv), q, cache, ctx, table, stride, s.window, s.scale,
-                                     softcap=s.score_softcap, slope_exponent=s.distance_slope_exponent, chunk=s.chunk)
+            if ((s.value_dim == s.head_dim and not special and out_scale == 1.0 and out.is_contiguous())
+                    or attention_backend.takes_changed_scores(self.dtype, nh, nkv, d, cache.page_size, dv)):
+                attention_backend.attend(heads_out, q, cache, ctx, table, stride, s.window, s.scale, softcap=s.score_softcap,
+                                         slope_exponent=s.distance_slope_exponent, chunk=s.chunk, sink=self.sink_scores,
+                                         keep_first=s.keep_first, out_scale=out_scale)
+                return
+        if special or self._changed_scores():
+            kernels.attention_plain(heads_out, q, cache["k"], cache["v"], ctx.positions, ctx.req_of_token, table, stride,
+                                    s.window, s.scale, ctx.err, sink=self.sink_scores, softcap=s.score_softcap,
+                                    slope_exponent=s.distance_slope_exponent, chunk=s.chunk, keep_first=s.keep_first,
+                                    out_scale=out_scale)
             return
         # queries per block: the longest portion decides (a step of single tokens takes one query per block
         # and cuts the keys instead); a replayed step must not look at its actual lengths
@@ -188,20 +231,14 @@ class TalkingAttention(Mixer):
         mma = (USE_TENSOR_CORES and self.dtype == torch.bfloat16 and out.stride(0) % 2 == 0 and out.data_ptr() % 4 == 0
                and kernels.attn_talking_mma_tile(nh, nkv, d, dv, longest) > 0)
         bq = kernels.attn_talking_mma_tile(nh, nkv, d, dv, longest) if mma else kernels.attn_talking_tile(nh, d, dv, longest)
-        if self._changed_scores():
-            if out_scale != 1.0 or not out.is_contiguous():
-                raise kernels.KernelError("attention with changed scores writes a contiguous, unscaled result")
-            kernels.attention_plain(out.view(T, nh, dv), q, cache["k"], cache["v"], ctx.positions, ctx.req_of_token, table,
-                                    stride, s.window, s.scale, ctx.err, softcap=s.score_softcap,
-                                    slope_exponent=s.distance_slope_exponent, chunk=s.chunk)
-            return
-        if bq <= 0 and not s.talking_heads and out_scale == 1.0 and out.is_contiguous():
+        if bq <= 0 and not s.talking_heads:
             # no mix across heads: a head needs no other head in its block, and the kernel with one warp per
             # (token, head) takes any number of heads of any size (a silent entry of score 0 is a sink of zeros)
             if s.sink and getattr(self, "_zero_sink", None) is None:
                 self._zero_sink = torch.zeros(nh, dtype=torch.float32, device=self.device)
-            kernels.attention_plain(out.view(T, nh, dv), q, cache["k"], cache["v"], ctx.positions, ctx.req_of_token, table,
-                                    stride, s.window, s.scale, ctx.err, sink=self._zero_sink if s.sink else None)
+            kernels.attention_plain(heads_out, q, cache["k"], cache["v"], ctx.positions, ctx.req_of_token, table,
+                                    stride, s.window, s.scale, ctx.err, sink=self._zero_sink if s.sink else None,
+                                    out_scale=out_scale)
             return
         if bq <= 0:
             raise kernels.KernelError(f"attention with {nh} heads of {d}/{dv} channels does not fit the kernel's tile")
