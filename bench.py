@@ -11,6 +11,7 @@
     python bench.py --compare gulipel [--size 1k|4k]        # the Gulipel design beside Tidarax at equal layer sizes
     python bench.py --compare mikutar [--size 1k|4k]        # the Mikutar design beside Dufitar at equal layer sizes
     python bench.py --compare napuzen [--size 1k|4k]        # the Napuzen design beside Dufitar and Gulipel at equal layer sizes
+    python bench.py --compare dalalix [--size 1k|4k]        # the Dalalix design beside Mikutar and Gulipel at equal layer sizes
 
 Prints ONE JSON line.  ``value`` is decoded tokens per second at batch 8 and the context length
 of the configuration (a "step" is one decode step of the whole batch), timed on the device with
@@ -326,6 +327,24 @@ def napuzen_config(z: dict, lat: dict, layers: int, vocab: int) -> dict:
                 layers=out)
 
 
+# --compare dalalix: convolved attention, attention with biases, attention beside a matrix memory, convolved attention;
+# experts in every layer, four groups of which two are kept; four residual streams; a window wider than the benchmark's
+# context that keeps the first 64 tokens; the memory with as many heads as the attention.
+def dalalix_config(z: dict, layers: int, vocab: int) -> dict:
+    d = z["head_dim"]
+    common = dict(heads=z["heads"], kv_heads=z["kv_heads"], dim=d, vdim=d, scale=d ** -0.5)
+    mlp = dict(kind="moe", expert=dict(ff=z["expert_ff"], limit=7.0),
+               router=dict(experts=z["experts"], top=z["top"], groups=dict(count=4, keep=2)))
+    conv = dict(type="attention", mixer=dict(common, conv=4), mlp=mlp)
+    biased = dict(type="attention_2", mixer=common, mlp=mlp)
+    left = dict(common, mask=dict(size=COMPARE_WINDOW, keep_first=64), rot=dict(dims=d // 2, base=500000.0))
+    par = dict(type="parallel", mlp=mlp, mixer=dict(left=left, left_scale=0.75, right_scale=0.5,
+                                                    right=dict(heads=z["heads"], dim=d, vdim=d, gate_cap=15.0)))
+    return dict(architecture="Dalalix", vocab=vocab, width=z["hidden"], norm=dict(eps=1e-6), streams=4, logit_softcap=30.0,
+                embedding=dict(bigram=dict(buckets=50021, mul_prev=8191, mul_cur=127)),
+                layers=[(conv, biased, par, conv)[i % 4] for i in range(layers)])
+
+
 def compare(args) -> int:
     """Prefill and decode throughput of a model of the named design and of a Qwen3 model of the same layer sizes
     (random weights, `--layers` layers each, default 4), then the design's kernels one by one beside their like
@@ -344,6 +363,8 @@ def compare(args) -> int:
     elif args.compare == "mikutar":     # its closest model is the other one with gated window attention and a float32 stream
         models = {"Mikutar": mikutar_config(z, L, V), "Mikutar, first layers twice": mikutar_config(z, L, V, loop=True),
                   "Dufitar": dufitar_config(z, LATENT_SIZES[args.size], L, V)}
+    elif args.compare == "dalalix":     # gated attention and experts as in Mikutar, a matrix state beside attention as in Gulipel
+        models = {"Dalalix": dalalix_config(z, L, V), "Mikutar": mikutar_config(z, L, V), "Gulipel": gulipel_config(z, L, V, ctx_len + 128)}
     elif args.compare == "napuzen":     # latent attention as in Dufitar, a recurrence with a matrix state as in Gulipel
         models = {"Napuzen": napuzen_config(z, LATENT_SIZES[args.size], L, V), "Dufitar": dufitar_config(z, LATENT_SIZES[args.size], L, V),
                   "Gulipel": gulipel_config(z, L, V, ctx_len + 128)}
@@ -400,6 +421,10 @@ def compare(args) -> int:
         records = measure.mikutar_kernels(hidden=z["hidden"], heads=z["heads"], kv_heads=z["kv_heads"], head_dim=z["head_dim"],
                                           intermediate=z["intermediate"], experts=z["experts"], expert_ff=z["expert_ff"],
                                           top=z["top"], hbm_gbs=pk["hbm_gbs"], peak_tflops=pk["bf16_tflops"])
+    elif args.compare == "dalalix":
+        records = measure.dalalix_kernels(hidden=z["hidden"], heads=z["heads"], kv_heads=z["kv_heads"], head_dim=z["head_dim"],
+                                          experts=z["experts"], expert_ff=z["expert_ff"], top=z["top"], hbm_gbs=pk["hbm_gbs"],
+                                          peak_tflops=pk["bf16_tflops"])
     elif args.compare == "napuzen":
         lat = LATENT_SIZES[args.size]
         records = measure.napuzen_kernels(hidden=z["hidden"], heads=z["heads"], head_dim=z["head_dim"], kv_rank=lat["kv_rank"],
@@ -446,9 +471,9 @@ def main() -> int:
                     help="with --kernels: the attention kernels alone at this head layout, over short and long contexts")
     ap.add_argument("--case", default="", metavar="decode:BATCHxCONTEXT | prefill:CACHED+NEW",
                     help="with --kernels --attn: this one case instead of the standard ones")
-    ap.add_argument("--compare", default="", choices=["", "tidarax", "dufitar", "gulipel", "mikutar", "napuzen"],
+    ap.add_argument("--compare", default="", choices=["", "tidarax", "dufitar", "gulipel", "mikutar", "napuzen", "dalalix"],
                     help="instead of the step benchmark: prefill and decode throughput of this design beside its closest model "
-                         "(Qwen3; for gulipel, Tidarax; for mikutar, Dufitar; for napuzen, Dufitar and Gulipel) at equal layer sizes, and its kernels beside their like kernels; one JSON line each")
+                         "(Qwen3; for gulipel, Tidarax; for mikutar, Dufitar; for napuzen, Dufitar and Gulipel; for dalalix, Mikutar and Gulipel) at equal layer sizes, and its kernels beside their like kernels; one JSON line each")
     ap.add_argument("--size", default="4k", choices=sorted(COMPARE_SIZES), help="layer sizes of --compare")
     ap.add_argument("--kernels", action="store_true",
                     help="instead of the step benchmark, time single kernels at serving sizes: one JSON line each")

@@ -59,12 +59,14 @@ def _attention_context(entries, page_size: int, device):
 
 def decode_attention(cases: Sequence = ((1, 4096), (8, 4096), (64, 4096), (8, 32768)), *, heads: int = 32,
                      kv_heads: int = 8, head_dim: int = 128, page_size: int = 16, hbm_gbs: float = 0.0,
-                     device="cuda:0", softcap=None, slope_exponent=None, chunk=None) -> List[Dict]:
+                     device="cuda:0", softcap=None, slope_exponent=None, chunk=None, window=None, keep_first: int = 0,
+                     sink=None) -> List[Dict]:
     """One decode token per request over `context` cached tokens, for (batch, context) cases.  ``softcap``,
-    ``slope_exponent``, ``chunk``: the attention with capped scores, a distance bias and a chunked mask."""
+    ``slope_exponent``, ``chunk``, ``window``, ``keep_first``, ``sink``: the attention with capped scores, a distance bias, a
+    chunked mask, a sliding window, first positions kept beside it and a sink (float32 per head)."""
     out = []
-    changes = dict(softcap=softcap, slope_exponent=slope_exponent, chunk=chunk)
-    mask = kernels.mask_code(None, chunk)
+    changes = dict(softcap=softcap, slope_exponent=slope_exponent, chunk=chunk, keep_first=keep_first, sink=sink)
+    mask = kernels.mask_code(window, chunk)
     for batch, context in cases:
         ctx, table, stride, num_pages = _attention_context([(context - 1, 1)] * batch, page_size, device)
         layers = 8 if batch * context <= 8 * 32768 else 2
@@ -73,16 +75,18 @@ def decode_attention(cases: Sequence = ((1, 4096), (8, 4096), (64, 4096), (8, 32
                   for _ in range(layers)]
         q = torch.randn(batch, heads, head_dim, device=device).bfloat16()
         o = torch.empty_like(q)
-        nbytes = batch * context * kv_heads * head_dim * 2 * 2
+        seen = context if not window else min(context, window + keep_first)
+        nbytes = batch * seen * kv_heads * head_dim * 2 * 2
         rec = {"kernel": "decode attention", "batch": batch, "context": context, "bytes": nbytes}
         for name, flag in (("tcgen05_us", True), ("mma_sync_us", False)):
             attention_backend.DECODE_TC = flag
             try:
                 # as in a step: the work is planned once, before the first kernel, for all layers
                 ctx.scratch.clear()
-                attention_backend.prepare_step(ctx, torch.bfloat16, heads, kv_heads, head_dim, page_size, mask, stride)
+                attention_backend.prepare_step(ctx, torch.bfloat16, heads, kv_heads, head_dim, page_size, mask, stride,
+                                               keep_first=keep_first)
                 torch.cuda.synchronize()   # the launches below run on a stream of their own
-                rec[name] = round(_graph_time_us(lambda: [attention_backend.attend(o, q, c, ctx, table, stride, None, head_dim ** -0.5,
+                rec[name] = round(_graph_time_us(lambda: [attention_backend.attend(o, q, c, ctx, table, stride, window, head_dim ** -0.5,
                                                                                    **changes)
                                                           for c in caches], layers), 1)
             finally:
@@ -98,19 +102,22 @@ def decode_attention(cases: Sequence = ((1, 4096), (8, 4096), (64, 4096), (8, 32
 
 def prefill_attention(cases: Sequence = ((0, 2048), (0, 8192), (24576, 8192)), *, heads: int = 32, kv_heads: int = 8,
                       head_dim: int = 128, page_size: int = 16, peak_tflops: float = 0.0, device="cuda:0", softcap=None,
-                      slope_exponent=None, chunk=None) -> List[Dict]:
+                      slope_exponent=None, chunk=None, window=None, keep_first: int = 0, sink=None) -> List[Dict]:
     """One request bringing `new` tokens after `cached` ones, for (cached, new) cases.  ``softcap``,
-    ``slope_exponent``, ``chunk``: the attention with capped scores, a distance bias and a chunked mask."""
+    ``slope_exponent``, ``chunk``, ``window``, ``keep_first``, ``sink``: as in ``decode_attention``."""
     out = []
-    changes = dict(softcap=softcap, slope_exponent=slope_exponent, chunk=chunk)
-    mask = kernels.mask_code(None, chunk)
+    changes = dict(softcap=softcap, slope_exponent=slope_exponent, chunk=chunk, keep_first=keep_first, sink=sink)
+    mask = kernels.mask_code(window, chunk)
     for cached, new in cases:
         ctx, table, stride, num_pages = _attention_context([(cached, new)], page_size, device)
         cache = LayerCache.of_keys_and_values(torch.randn(num_pages, kv_heads, page_size, head_dim, device=device).bfloat16(),
                            torch.randn(num_pages, kv_heads, page_size, head_dim, device=device).bfloat16(), 0, page_size)
         q = torch.randn(new, heads, head_dim, device=device).bfloat16()
         o = torch.empty_like(q)
-        flops = 4.0 * heads * head_dim * (new * cached + new * (new + 1) / 2)
+        seen = np.arange(cached + 1, cached + new + 1, dtype=np.float64)
+        if window:
+            seen = np.minimum(seen, window + keep_first)
+        flops = 4.0 * heads * head_dim * float(seen.sum())
         rec = {"kernel": "prefill attention", "cached": cached, "new": new, "flops": flops}
         for name, flag in (("tcgen05_us", True), ("mma_sync_us", False)):
             attention_backend.PREFILL_TC = flag
@@ -118,9 +125,10 @@ def prefill_attention(cases: Sequence = ((0, 2048), (0, 8192), (24576, 8192)), *
                 # several launches replayed from a CUDA graph: the host's share of a launch (tensor maps, wrappers)
                 # is not in the time, as it is not in a step, where launches queue ahead of the device
                 per = 4 if new * (cached + new) <= 8192 * 16384 else 1
-                attention_backend.prepare_step(ctx, torch.bfloat16, heads, kv_heads, head_dim, page_size, mask, stride)
+                attention_backend.prepare_step(ctx, torch.bfloat16, heads, kv_heads, head_dim, page_size, mask, stride,
+                                               keep_first=keep_first)
                 torch.cuda.synchronize()
-                rec[name] = round(_graph_time_us(lambda: [attention_backend.attend(o, q, cache, ctx, table, stride, None, head_dim ** -0.5,
+                rec[name] = round(_graph_time_us(lambda: [attention_backend.attend(o, q, cache, ctx, table, stride, window, head_dim ** -0.5,
                                                                                    **changes)
                                                           for _ in range(per)], per), 1)
             finally:
@@ -989,6 +997,162 @@ def napuzen_kernels(*, hidden: int = 4096, heads: int = 32, head_dim: int = 128,
                    lambda i: kernels.expert_select_gate(a2[i], g2[i], choice, None, None, rq, top, E, err, weights=weight,
                                                         activation="swish_clamp", params=(7.0, 1.702)), tokens=T)
             del gus, acts, g2, a2
+    if int(err):
+        raise RuntimeError("a kernel reported an error: " + kernels.describe_error(int(err)))
+    return out
+
+
+def dalalix_kernels(*, hidden: int = 4096, heads: int = 32, kv_heads: int = 8, head_dim: int = 128, streams: int = 4,
+                    conv: int = 4, experts: int = 8, expert_ff: int = 3072, top: int = 2, tokens: int = 2048,
+                    decode: Sequence[int] = (8, 4096), page_size: int = 16, hbm_gbs: float = 0.0, peak_tflops: float = 0.0,
+                    device="cuda:0") -> List[Dict]:
+    """One record per kernel of the Dalalix path: time, bytes and the share of its floor (the bytes that must cross
+    memory at the measured copy rate; for the scan also its arithmetic at the nominal FMA rate, for the attention its
+    products at the measured matrix-product peak), each followed by the like kernel of the design it is closest to,
+    measured the same way ("like: ...")."""
+    out: List[Dict] = []
+    err = torch.zeros(1, dtype=torch.int32, device=device)
+    sets = 4
+    f32 = lambda *shape: torch.randn(*shape, device=device)
+    bf = lambda *shape: torch.randn(*shape, device=device).bfloat16()
+    i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=device)
+
+    def record(name, nbytes, run, flops=0.0, n=sets, **more):
+        us = _graph_time_us(lambda: [run(i) for i in range(n)], n)
+        floor_us = max(nbytes / (hbm_gbs or 6650.0) / 1e3, flops / FP32_FMA_TFLOPS_NOMINAL / 1e6)
+        out.append(dict({"kernel": name, "bytes": nbytes, "us": round(us, 1), "gbs": round(nbytes / us / 1e3, 1),
+                         "floor_us": round(floor_us, 2), "frac_of_floor": round(floor_us / us, 3)}, **more))
+
+    H, G, d, C, n_s = heads, kv_heads, head_dim, hidden, streams
+    B, context = decode
+    steps = (("a prompt", tokens, i32([0, tokens]), i32([0]), torch.zeros(tokens, dtype=torch.int32, device=device), 1),
+             ("single tokens", B, i32(list(range(B + 1))), i32(list(range(B))), i32(list(range(B))), B))
+
+    # attention: a window that keeps the first tokens and a sink, beside the engine's attention as it is
+    sink = f32(H)
+    for name, kw in ((f"window {tokens // 2} that keeps 64 + sink", dict(window=tokens // 2, keep_first=64, sink=sink)),
+                     (f"window {2 * context} that keeps 64 + sink", dict(window=2 * context, keep_first=64, sink=sink)),
+                     (f"like: the engine's attention, window {tokens // 2}", dict(window=tokens // 2)),
+                     ("like: the engine's attention, every earlier key", {})):
+        rec = prefill_attention(((0, tokens),), heads=H, kv_heads=G, head_dim=d, page_size=page_size, peak_tflops=peak_tflops, **kw)[0]
+        out.append({"kernel": "prompt attention (tcgen05), " + name, "tokens": tokens, "us": rec["tcgen05_us"],
+                    "tensor_tflops": rec["tflops"], "frac_of_floor": rec.get("frac_of_peak")})
+        rec = decode_attention(((B, context),), heads=H, kv_heads=G, head_dim=d, page_size=page_size, hbm_gbs=hbm_gbs, **kw)[0]
+        out.append({"kernel": "single-token attention (tcgen05), " + name, "batch": B, "context": context,
+                    "us": rec["tcgen05_us"], "gbs": rec["gbs"], "frac_of_floor": rec.get("frac_of_hbm")})
+
+    # the residual streams: write to all, read their weighted sum, norm
+    w, w2, gain = f32(C), f32(C), f32(C)
+    r_, m_, w_ = f32(n_s), f32(n_s, n_s) * 0.3, f32(n_s)
+    for what, T, qs, sl, rq, ne in steps:
+        xs = [f32(T, n_s, C) for _ in range(sets)]
+        bs = [f32(T, C) for _ in range(sets)]
+        hs = [torch.empty(T, C, dtype=torch.bfloat16, device=device) for _ in range(sets)]
+        record(f"{n_s} residual streams: mixed and written, read and normed, {what}", T * C * (8 * n_s + 6),
+               lambda i: kernels.stream_mix(hs[i], xs[i], r_, w, 1e-6, err, branch=bs[i], mix=m_, write=w_, x_out=xs[i]), tokens=T)
+        del xs
+        x1 = [f32(T, C) for _ in range(sets)]
+        record(f"like: Mikutar float32 residual sum + RMS norm, {what}", T * C * 14,
+               lambda i: kernels.rmsnorm(hs[i], x1[i], w, 1e-6, err, branch=bs[i], sum_out=x1[i]), tokens=T)
+        record(f"like: Gulipel normed branch x learned scale + float32 sum + norm, {what}", T * C * 14,
+               lambda i: kernels.rms_chain(hs[i], x1[i], w, 1e-6, err, branch=bs[i], branch_weight=w2, branch_eps=1e-6, gain=gain,
+                                           sum_out=x1[i]), tokens=T)
+        del x1, bs, hs
+
+    # queries, keys and values: convolution + value norm + page write; biases + rotation of halves + page write
+    C3 = (H + 2 * G) * d
+    for what, T, qs, sl, rq, ne in steps:
+        pages = (T + page_size - 1) // page_size if ne == 1 else ne
+        stride = pages if ne == 1 else 1
+        pos = torch.arange(T, dtype=torch.int32, device=device) if ne == 1 else i32([5] * T)
+        tab = torch.randperm(pages, device=device).to(torch.int32)
+        qo = [torch.empty(T, H, d, dtype=torch.bfloat16, device=device) for _ in range(sets)]
+        kcs = [torch.zeros(pages, G, page_size, d, dtype=torch.bfloat16, device=device) for _ in range(sets)]
+        vcs = [torch.zeros_like(k) for k in kcs]
+        rows = [bf(T, C3 + H * d) for _ in range(sets)]
+        states = [torch.zeros(ne, conv - 1, C3, dtype=torch.bfloat16, device=device) for _ in range(sets)]
+        taps = f32(conv, C3)
+        record(f"convolution of {conv} taps on q, k and v + value norm + cache write, {what}",
+               T * C3 * 4 + 2 * ne * (conv - 1) * C3 * 2,
+               lambda i: kernels.qkv_prepare(qo[i], kcs[i], vcs[i], rows[i], None, None, None, pos, rq, tab, stride, H, G, d, d, 0, False,
+                                             0, 1e-6, True, err, row_len=C3 + H * d, conv=(taps, states[i], qs, sl, ne > 1),
+                                             value_eps=1e-6), tokens=T)
+        inv, bias = torch.rand(d // 4, device=device), f32(C3)
+        dense = [bf(T, C3) for _ in range(sets)]
+        record(f"biases + rotation of halves + cache write, {what}", T * C3 * 4,
+               lambda i: kernels.qkv_prepare(qo[i], kcs[i], vcs[i], dense[i], None, None, inv, pos, rq, tab, stride, H, G, d, d, d // 2,
+                                             False, 0, 1e-6, True, err, bias=bias), tokens=T)
+        record(f"biases + cache write, {what}", T * C3 * 4,
+               lambda i: kernels.qkv_prepare(qo[i], kcs[i], vcs[i], dense[i], None, None, None, pos, rq, tab, stride, H, G, d, d, 0,
+                                             False, 0, 1e-6, True, err, bias=bias), tokens=T)
+        qw, kw_ = f32(d), f32(d)
+        record(f"like: Gulipel biases + norm per head + cache write, {what}", T * C3 * 4,
+               lambda i: kernels.qkv_prepare(qo[i], kcs[i], vcs[i], dense[i], qw, kw_, None, pos, rq, tab, stride, H, G, d, d, 0,
+                                             False, 1, 1e-6, True, err, bias=bias), tokens=T)
+        # (a convolution on its own, as the recurrent layers of Gulipel run it: float32 in and out, with SiLU)
+        us, ys = [f32(T, C3) for _ in range(sets)], [torch.empty(T, C3, device=device) for _ in range(sets)]
+        fst, tp = [torch.zeros(ne, conv - 1, C3, device=device) for _ in range(sets)], taps.t().contiguous()
+        record(f"like: Gulipel convolution of {conv} taps + SiLU, {what}", T * C3 * 8 + 2 * ne * (conv - 1) * C3 * 4,
+               lambda i: kernels.conv_silu(ys[i], us[i], 0, tp, None, fst[i], rq, qs, sl, ne), tokens=T)
+        inns = [bf(T, H * d) for _ in range(sets)]
+        record(f"sigmoid gate per channel (in place), {what}", 3 * T * H * d * 2,
+               lambda i: kernels.gate_sigmoid(inns[i], inns[i].view(T, H, d).transpose(0, 1), rows[i][:, C3:]), tokens=T)
+        del qo, kcs, vcs, rows, states, dense, us, ys, fst, inns
+
+    # the matrix memory beside the recurrences with a matrix state
+    qk = H * d
+    for what, T, qs, sl, rq, ne in steps:
+        projs = [f32(T, 4 * qk + 2 * H) for _ in range(sets)]
+        os_ = [torch.empty(T, qk, device=device) for _ in range(sets)]
+        divs = [torch.empty(T, H, device=device) for _ in range(sets)]
+        gated = [torch.empty(T, 2 * qk, dtype=torch.bfloat16, device=device)[:, qk:] for _ in range(sets)]
+        sts = [dict(S=torch.zeros(ne, H, d, d, device=device), n=torch.zeros(ne, H, d, device=device),
+                    m=torch.zeros(ne, H, 2, 2, device=device)) for _ in range(sets)]
+        start = i32([0] * ne)
+        b1, b2, nw, nw1 = f32(H), f32(H) + 3.0, f32(qk), f32(d)
+        record(f"matrix memory scan, {what}", T * 4 * qk * 4 + 2 * ne * qk * d * 4,
+               lambda i: kernels.matrix_memory(os_[i], divs[i], projs[i], 4 * qk, b1, b2, 15.0, sts[i], qs, start, sl, ne, H, d, d,
+                                               d ** -0.5, 1e-6), flops=6.0 * T * qk * d, tokens=T, heads=H, dim=d)
+        record(f"division + norm per head + sigmoid gate, {what}", T * qk * 10,
+               lambda i: kernels.gated_head_norm(gated[i], os_[i], projs[i], 3 * qk, nw, d, 1e-6, gate_after=True, div=divs[i],
+                                                 out_scale=0.5), tokens=T)
+        alphas = [torch.rand(T, qk, device=device) for _ in range(sets)]
+        record(f"like: Napuzen linear attention scan, {what}", T * 5 * qk * 4 + 2 * ne * qk * d * 4,
+               lambda i: kernels.linear_scan(os_[i], projs[i], alphas[i], sts[i]["S"], qs, sl, ne, H, d, d, d ** -0.5),
+               flops=6.0 * T * qk * d, tokens=T, heads=H, dim=d)
+        qkvs, ags = [f32(T, 3 * qk) for _ in range(sets)], [f32(T, 2 * qk) for _ in range(sets)]
+        alog, bd = f32(H), f32(qk)
+        record(f"like: Gulipel gated delta rule, {what}", T * (6 * qk + H) * 4 + 2 * ne * qk * d * 4,
+               lambda i: kernels.delta_rule(os_[i], qkvs[i], projs[i], 3 * qk, ags[i], bd, alog, sts[i]["S"], qs, sl, ne, H, H, d, d),
+               flops=8.0 * T * qk * d, tokens=T, heads=H, dim=d)
+        whole = [torch.empty(T, qk, dtype=torch.bfloat16, device=device) for _ in range(sets)]
+        record(f"like: Gulipel norm per head + sigmoid gate, {what}", T * qk * 10,
+               lambda i: kernels.gated_head_norm(whole[i], os_[i], ags[i], qk, nw1, d, 1e-6, gate_after=True), tokens=T)
+        del projs, os_, divs, gated, sts, alphas, qkvs, ags, whole
+
+    # router and experts
+    E, Fi = experts, expert_ff
+    wr, corr = f32(E, C) * C ** -0.5, f32(E) * 0.3
+    for what, T, qs, sl, rq, ne in steps:
+        hs = [bf(T, C) for _ in range(sets)]
+        choice, weight = torch.zeros(T, top, dtype=torch.int32, device=device), torch.zeros(T, top, device=device)
+        record(f"softmax router with groups, {what}", T * C * 2 + E * C * 4,
+               lambda i: kernels.expert_router(choice, weight, hs[i], wr, None, rq, top, 4, 2, 1, renormalize=True, softmax=True,
+                                               renormalize_eps=1e-20), tokens=T)
+        record(f"like: Mikutar sigmoid router with groups, {what}", T * C * 2 + E * C * 4,
+               lambda i: kernels.expert_router(choice, weight, hs[i], wr, corr, rq, top, 4, 2, 2), tokens=T)
+        if T == tokens:
+            nrows = T * top
+            offsets, perm, inv_ = i32([0] * (E + 1)), i32([0] * nrows), i32([0] * nrows)
+            kernels.expert_route(offsets, perm, inv_, choice, None, None, rq, T, top, E, err)
+            ys, outs = [f32(nrows, C) for _ in range(sets)], [torch.empty(T, C, device=device) for _ in range(sets)]
+            bases = [f32(T, C) for _ in range(sets)]
+            record(f"experts' weighted sum, {what}", T * C * 4 * (top + 1),
+                   lambda i: kernels.expert_combine(outs[i], ys[i], inv_, top, weights=weight), tokens=T)
+            record(f"like: Mikutar experts' weighted sum onto the shared expert, {what}", T * C * 4 * (top + 2),
+                   lambda i: kernels.expert_combine(outs[i], ys[i], inv_, top, weights=weight, base=bases[i]), tokens=T)
+            del ys, outs, bases
+        del hs
     if int(err):
         raise RuntimeError("a kernel reported an error: " + kernels.describe_error(int(err)))
     return out
