@@ -7,12 +7,12 @@ import numpy as np
 from xinfer_b200.native import host_lib
 
 
-def work_list(counts, starts, dec_max, window, 0, heads, kv_heads, max_ctas):
+def work_list(counts, starts, dec_max, window, heads, kv_heads, max_ctas, keep=0):
     counts, starts = np.asarray(counts, dtype=np.int32), np.asarray(starts, dtype=np.int32)
     cap = max_ctas + 1 + 4 * int(((counts + 127) // 128).sum()) * heads + 8
     out = np.full(cap, -9, dtype=np.int32)
     ctas = ctypes.c_int(0)
-    used = host_lib().xb_attn_prefill_work(len(counts), counts.ctypes.data, starts.ctypes.data, dec_max, window, 0, heads, kv_heads,
+    used = host_lib().xb_attn_prefill_work(len(counts), counts.ctypes.data, starts.ctypes.data, dec_max, window, keep, heads, kv_heads,
                                            max_ctas, out.ctypes.data, cap, ctypes.byref(ctas))
     c = ctas.value
     offs = out[: c + 1]
@@ -69,3 +69,14 @@ def test_nothing_to_do_and_too_small_a_buffer():
     ctas = ctypes.c_int(0)
     assert host_lib().xb_attn_prefill_work(1, counts.ctypes.data, starts.ctypes.data, 4, 0, 0, 8, 2, 148, out.ctypes.data, 10,
                                            ctypes.byref(ctas)) == -1
+
+
+def test_tiles_of_kept_first_positions_count_once():
+    """Four portions whose windows lie far back, just behind and over the first positions that stay visible: the
+    longest portion by its tiles, kept ones included, comes first."""
+    counts, window = [64, 64, 64, 64], 64
+    starts = [10000, 128, 64, 0]
+    # tiles of the window alone, and with 130 kept positions (three tiles, as far as they lie before the window's)
+    for keep, tiles in ((0, [2, 2, 2, 1]), (130, [5, 3, 2, 1])):
+        _, offs, items, _ = work_list(counts, starts, 4, window, 1, 1, 1, keep)
+        assert [int(b) for b in items[:, 0]] == sorted(range(4), key=lambda b: -tiles[b])

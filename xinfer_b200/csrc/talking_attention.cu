@@ -28,10 +28,10 @@
 // With CONV every channel of the row first passes a causal convolution over time, y_t = sum_j taps[j, c] u_(t-K+1+j),c
 // (taps [K, channels], no bias): the K-1 rows before a step's first token of a request come from conv_state[slot]
 // ([K-1, channels], oldest first, in the rows' own type), the others from the rows of this step.  keep_state: every
-// request brings one token, and the block that has read its old rows leaves the last K-1 there.
+// request brings one token, and the warp that has read a head's old rows leaves the last K-1 there.
 // value_eps >= 0: a value head is divided by its root mean square (this eps under the root) before it is cached.
 // q goes to q_out[t, h], k and v into their pages ([page, kv_head, slot, d] and [.., dv]).
-// One block per token, one warp per head at a time; the angles' cos/sin are formed once per token.
+// One block per token (few tokens: several), one warp per head at a time; the angles' cos/sin are formed once per token.
 // ------------------------------------------------------------------------------------------
 // Four consecutive elements at once where the row allows it (bfloat16: 8-byte accesses; float32: 16-byte).
 template <typename T>
@@ -179,7 +179,8 @@ __global__ void qkv_prepare_kernel(T* __restrict__ q_out, T* __restrict__ k_cach
     }
     // the query's temperature: it grows with the logarithm of the number of whole periods the sequence has seen
     const float q_mul = temp_every > 0 ? 1.f + temp_coef * logf((float)((pos + 1) / temp_every) + 1.f) : 1.f;
-    for (int h = warp; h < nh + 2 * nkv; h += nwarps) {
+    const int h_first = blockIdx.y * nwarps + warp, h_step = gridDim.y * nwarps;      // the heads of this warp
+    for (int h = h_first; h < nh + 2 * nkv; h += h_step) {
         if (h >= nh + nkv) {      // a value head: copy (plus its bias)
             if (kv_row < 0) continue;
             const int g = h - nh - nkv;
@@ -341,11 +342,26 @@ __global__ void qkv_prepare_kernel(T* __restrict__ q_out, T* __restrict__ k_cach
         __syncwarp();
     }
     if (CONV && keep_state && slot >= 0 && K > 1) {
-        __syncthreads();        // every warp has read the old rows
+        __syncwarp();           // this warp has read the old rows of its heads' channels, and nobody else reads them
         T* st = conv_state + (size_t)slot * (K - 1) * C;
-        for (int c = threadIdx.x; c < C; c += blockDim.x) {
-            for (int j = 0; j + 1 < K - 1; ++j) st[(size_t)j * C + c] = st[(size_t)(j + 1) * C + c];
-            st[(size_t)(K - 2) * C + c] = row[c];
+        for (int h = h_first; h < nh + 2 * nkv; h += h_step) {
+            const int c0 = h < nh + nkv ? h * d : (nh + nkv) * d + (h - nh - nkv) * dv, len = h < nh + nkv ? d : dv;
+            if (vec4) {
+                for (int c = c0 + lane * 4; c < c0 + len; c += 128) {
+                    float v[4];
+                    for (int j = 0; j + 1 < K - 1; ++j) {
+                        load4<T>(st + (size_t)(j + 1) * C + c, v);
+                        store4<T>(st + (size_t)j * C + c, v);
+                    }
+                    load4<T>(row + c, v);
+                    store4<T>(st + (size_t)(K - 2) * C + c, v);
+                }
+            } else {
+                for (int c = c0 + lane; c < c0 + len; c += 32) {
+                    for (int j = 0; j + 1 < K - 1; ++j) st[(size_t)j * C + c] = st[(size_t)(j + 1) * C + c];
+                    st[(size_t)(K - 2) * C + c] = row[c];
+                }
+            }
         }
     }
 }
@@ -365,6 +381,12 @@ XB_EXPORT int xb_qkv_prepare(int dtype, void* q_out, void* k_cache, void* v_cach
     // a warp per head at a time: as many warps as a token has heads, up to 16
     const int heads = nh + 2 * nkv;
     int threads = heads >= 16 ? 512 : (heads >= 8 ? 256 : 128);
+    // few tokens: four heads per block, so that they spread over the machine (one norm over a whole projection: one block)
+    unsigned spread = 1;
+    if (tokens <= 64 && norm_mode != 3) {
+        threads = 128;
+        spread = (unsigned)((heads + 3) / 4);
+    }
     const int wide = value_eps >= 0.f && dv > d ? dv : d;
     size_t smem = ((size_t)rot + (size_t)(threads / 32) * wide) * sizeof(float);
     while (smem > 48 * 1024 && threads > 32) {     // very wide heads: fewer warps, each still with room for its head
@@ -378,7 +400,7 @@ XB_EXPORT int xb_qkv_prepare(int dtype, void* q_out, void* k_cache, void* v_cach
                       !((uintptr_t)taps & 15) && !((uintptr_t)conv_state & (4 * esz - 1)) && !(((uintptr_t)bias | (uintptr_t)q_w | (uintptr_t)k_w) & 15) &&
                       !(((uintptr_t)qkv | (uintptr_t)q_out | (uintptr_t)k_cache | (uintptr_t)v_cache) & (4 * esz - 1))) ? 1 : 0;
 #define XB_PREPARE(T, CONV)                                                                                               \
-    qkv_prepare_kernel<T, CONV><<<tokens, threads, smem, stream>>>(                                                      \
+    qkv_prepare_kernel<T, CONV><<<dim3(tokens, spread), threads, smem, stream>>>(                                                      \
         (T*)q_out, (T*)k_cache, (T*)v_cache, (const T*)qkv, q_w, k_w, inv_freq, positions, req_of_token, block_table,    \
         table_stride, nh, nkv, d, dv, rot, interleaved, norm_mode, page_size, num_pages, eps, write_kv, vec4, rot_mag,   \
         bias, temp_coef, temp_every, row_len, v_off, taps, K, (T*)conv_state, q_start, slots, keep_state, value_eps, err)
