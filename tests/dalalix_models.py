@@ -81,13 +81,20 @@ _D = [_again(_D, 2)] + [dict(l) for l in _D]
 _D[0]["weights_of"] = 3
 _D += [dict(_D[2], weights_of=2)]
 
+# every router gives a token all its experts: nothing to decide, so that rounding never leads to another computation
+_F = [_moe(_parallel((4, 2, 32, 32, 0.2), 40, 20, (16, 2000.0), (4, 16, 16), 15.0, (1.0, 0.5)), 24, 1.2, 4, 4, (2, 2)),
+      _moe(_conv(4, 1, 32, 48, 0.15, 4), 32, 3.0, 2, 2),
+      _biased(4, 2, 64, 64, 0.1)]
+_F += [_again(_F, 0)]
+
 # name -> (config, seed, page size)
 TINY_D: Dict[str, tuple] = {
-    "A": (_cfg(83, 48, 1e-5, 3, _A, bigram=(37, 11, 5), softcap=9.0), 61, 8),
-    "B": (_cfg(157, 64, 3e-6, 4, _B, bigram=(210, 13, 150), softcap=30.0), 62, 16),
-    "C": (_cfg(120, 96, 1e-6, 1, _C), 63, 32),
-    "D": (_cfg(61, 52, 2e-6, 5, _D, bigram=(1, 3, 0), softcap=4.0), 64, 16),
+    "A": (_cfg(83, 48, 2e-2, 3, _A, bigram=(37, 11, 5), softcap=9.0), 61, 8),
+    "B": (_cfg(157, 64, 5e-2, 4, _B, bigram=(210, 13, 150), softcap=30.0), 62, 16),
+    "C": (_cfg(120, 96, 1e-2, 1, _C), 63, 32),
+    "D": (_cfg(61, 52, 3e-2, 5, _D, bigram=(1, 3, 0), softcap=4.0), 64, 16),
     "E": (_cfg(70, 40, 1e-5, 9, _A[:2], bigram=(64, 0, 1)), 65, 16),
+    "F": (_cfg(131, 64, 2e-2, 4, _F, bigram=(99, 5, 17), softcap=12.0), 66, 16),
 }
 
 

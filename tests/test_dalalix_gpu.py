@@ -13,6 +13,17 @@ from helpers import build_all_modes, replay_with_routes, row_error, run_trace
 pytestmark = pytest.mark.gpu
 
 DEV = "cuda:0"
+
+
+@pytest.fixture(autouse=True)
+def _one_thread():
+    """The plain implementation works on small matrices: threads would only wait for each other."""
+    n = torch.get_num_threads()
+    torch.set_num_threads(1)
+    yield
+    torch.set_num_threads(n)
+
+
 F64 = torch.float64
 
 
@@ -111,7 +122,7 @@ def _prepare_steps(H, G, d, dv, K, lens, cuts, dtype, seed, value_eps=1e-5, ps=8
     rows = [_rand(n, C, seed=seed + i).to(dtype) for i, n in enumerate(lens)]
     taps = _rand(C, K, seed=seed + 90, scale=0.6).float()
     R = len(lens)
-    slots = [(2 * i + 1) % (R + 1) for i in range(R)]
+    slots = [R - i for i in range(R)]
     state = torch.full((R + 1, max(K - 1, 1), C), 3.0, dtype=dtype, device=DEV)
     for s in slots:
         state[s].zero_()
@@ -599,7 +610,7 @@ def test_routed_experts_part_equals_plain(dtype, T, E, top, groups, keep, limit)
 # ---------------------------------------------------------------------------------------------
 # whole models: every way of cutting, pages and slots used again, layer by layer, generation
 # ---------------------------------------------------------------------------------------------
-LENGTHS = {"A": [70, 45, 130, 33], "B": [97, 41, 260, 150], "C": [170, 1, 75, 58], "D": [90, 2, 51, 140], "E": [40, 21, 70]}
+LENGTHS = {"A": [70, 45, 130, 33], "B": [97, 41, 260, 150], "C": [170, 1, 75, 58], "D": [90, 2, 51, 140], "E": [40, 21, 70], "F": [60, 31, 85]}
 
 
 def _tolerance(dtype, ref, cfg=None, w=None, p=None, routes=None):
@@ -826,7 +837,7 @@ def test_greedy_generation_in_float32_equals_plain(name, tmp_path):
 
 
 @pytest.mark.parametrize("graphs", [False, True], ids=["launched", "cuda_graph"])
-@pytest.mark.parametrize("name", ["B", "D"])
+@pytest.mark.parametrize("name", ["F"])
 def test_long_greedy_decoding_in_bfloat16_follows_the_plain_logits(name, graphs, tmp_path):
     """Each generated token is checked against the plain logits of the sequence the engine produced (bfloat16 may flip a
     near-tie): it must be the best token up to the drift.  Long enough for many pages per request and for windows to pass
@@ -843,7 +854,7 @@ def test_long_greedy_decoding_in_bfloat16_follows_the_plain_logits(name, graphs,
         seq = p + o.decode_output
         ref = plain.forward(cfg, w, seq)
         slack = 2 * 3.0 * float((plain.forward(cfg, w, seq, round_to=torch.bfloat16) - ref).abs().max())
-        assert slack < 0.5 * float(ref.max() - ref.min()), "the drift is too large for this to show anything"
+        assert slack < 0.2 * float(ref.max() - ref.min()), "the drift is too large for this to show anything"
         for i, tok in enumerate(o.decode_output):
             row = ref[len(p) + i - 1]
             assert row[tok] >= row.max() - slack, (i, tok)
@@ -853,8 +864,8 @@ def test_a_replayed_decode_step_equals_a_launched_one(tmp_path):
     """A CUDA graph is captured by running the step for real a few times; the memories, the convolutions' inputs and the
     token before go back to what they were."""
     from xinfer_b200 import SamplingParams
-    folder = make_folder(str(tmp_path / "model"), "B", torch.bfloat16)
-    ps = prompts("B", [7, 33, 18])
+    folder = make_folder(str(tmp_path / "model"), "F", torch.bfloat16)
+    ps = prompts("F", [7, 33, 18])
     outs = []
     for graphs in (False, True):
         eng = _engine(folder, "bf16", 16, disable_cuda_graph=not graphs)

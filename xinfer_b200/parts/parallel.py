@@ -48,8 +48,7 @@ class ParallelMixer(Mixer):
         return out
 
     def children(self):
-        # with one output product for both sides the combined matrix is this part's, else every side has its own
-        return (self.left, self.right) if self.spec.out_norms is not None else ()
+        return (self.left, self.right)
 
     def load(self, store) -> None:
         self.left.load(store)
@@ -59,6 +58,11 @@ class ParallelMixer(Mixer):
                                         for n in self.spec.out_norms)
             return
         self.w_o = torch.cat([self.left.output_weight(), self.right.output_weight()], dim=1).contiguous()
+        # the sides' own matrices are column ranges of it from here on (held once)
+        at = 0
+        for m in (self.left, self.right):
+            m.w_o = self.w_o[:, at:at + m.inner_width()]
+            at += m.inner_width()
 
     def cache_need(self):
         return self.left.cache_need() or self.right.cache_need()
