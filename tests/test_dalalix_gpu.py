@@ -185,10 +185,27 @@ def test_convolved_projections_however_the_tokens_are_cut(H, G, d, dv, K, dtype)
                 assert (a - b).abs().max() <= (1e-5 if dtype == torch.float32 else 1e-2) * (1 + b.abs().max())
 
 
-def test_convolution_without_a_value_norm_and_over_many_tokens():
-    got, want = _prepare_steps(4, 2, 16, 16, 4, [700, 3, 1, 130], [[(0, 700), (1, 3), (2, 1), (3, 130)]], torch.float32, 7, value_eps=None)
-    for g, w in zip(got, want):
-        assert all((a - b).abs().max() <= 1e-5 * (1 + b.abs().max()) for a, b in zip(g, w))
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+@pytest.mark.parametrize("H,G,d,dv,K", [(4, 2, 16, 16, 4), (3, 1, 200, 132, 3), (2, 2, 64, 180, 6), (5, 1, 96, 32, 1), (2, 1, 128, 128, 2),
+                                        (1, 1, 32, 260, 4), (2, 1, 16, 16, 9)])
+@pytest.mark.parametrize("value_eps", [None, 1e-5])
+def test_convolution_over_steps_of_many_tokens(H, G, d, dv, K, value_eps, dtype):
+    """Warps then take runs of tokens that cross from one request into the next and start in the middle of one; a request
+    goes on from a step of single tokens and from a portion shorter than the taps."""
+    lens = [700, 3, 1, 130]
+    for cuts in ([[(0, 700), (1, 3), (2, 1), (3, 130)]],
+                 [[(0, 2), (3, 1)], [(0, 90), (1, 1), (3, 2)], [(0, 1), (3, 1)], [(0, 607), (1, 2), (2, 1), (3, 126)]]):
+        got, want = _prepare_steps(H, G, d, dv, K, lens, cuts, dtype, 7, value_eps=value_eps)
+        for g, w in zip(got, want):
+            assert all((a - b).abs().max() <= (1e-5 if dtype == torch.float32 else 1e-2) * (1 + b.abs().max()) for a, b in zip(g, w))
+
+
+def test_both_forms_of_the_convolution_give_the_same_bits():
+    """Steps of more than 64 tokens take the form in runs, shorter ones a block per token."""
+    for dtype in (torch.float32, torch.bfloat16):
+        a, _ = _prepare_steps(4, 2, 32, 48, 4, [130], [[(0, 130)]], dtype, 11)
+        b, _ = _prepare_steps(4, 2, 32, 48, 4, [130], [[(0, 60)], [(0, 60)], [(0, 10)]], dtype, 11)
+        assert all(torch.equal(x, y) for x, y in zip(a[0], b[0]))
 
 
 def test_a_convolution_takes_no_biases():

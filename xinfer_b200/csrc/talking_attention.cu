@@ -366,6 +366,146 @@ __global__ void qkv_prepare_kernel(T* __restrict__ q_out, T* __restrict__ k_cach
     }
 }
 
+// The same for steps of many tokens where a head needs nothing but its convolution (and a value head its root mean
+// square): no rotation, no norm of q or k.  A warp takes one head and a run of tokens, its lanes four channels each (NV times
+// 128 per head); the K-1 rows before a token stay in registers and move along, so every row crosses memory once per run
+// (and K-1 of them twice).  Taps are added in the same order as above: both give the same bits.
+template <typename T, int K, int NV>
+__global__ void __launch_bounds__(256) qkv_conv_runs_kernel(T* __restrict__ q_out, T* __restrict__ k_cache, T* __restrict__ v_cache,
+                                                            const T* __restrict__ qkv, long long row_len,
+                                                            const float* __restrict__ taps, const T* __restrict__ conv_state,
+                                                            const int* __restrict__ positions, const int* __restrict__ req_of_token,
+                                                            const int* __restrict__ block_table, int table_stride,
+                                                            const int* __restrict__ q_start, const int* __restrict__ slots,
+                                                            int nh, int nkv, int d, int dv, int ps, int num_pages, float value_eps,
+                                                            int write_kv, int tokens, int run, int* err) {
+    const int lane = threadIdx.x & 31, h = blockIdx.y * (blockDim.x >> 5) + (threadIdx.x >> 5);
+    if (h >= nh + 2 * nkv) return;
+    const bool is_q = h < nh, is_v = h >= nh + nkv;
+    if (!is_q && !write_kv) return;
+    const int len = is_v ? dv : d, C = (nh + nkv) * d + nkv * dv;
+    const int col = is_v ? (nh + nkv) * d + (h - nh - nkv) * dv : h * d;
+    const int g = is_v ? h - nh - nkv : h - nh;       // (of a key or value head)
+    T* const cache = is_v ? v_cache : k_cache;
+    const bool unit = is_v && value_eps >= 0.f;
+    float tap[K][NV][4], win[K > 1 ? K - 1 : 1][NV][4];
+    bool in[NV];
+#pragma unroll
+    for (int e = 0; e < NV; ++e) {
+        const int c = lane * 4 + 128 * e;
+        in[e] = c < len;
+#pragma unroll
+        for (int j = 0; j < K; ++j) {
+            const float4 w4 = in[e] ? *reinterpret_cast<const float4*>(taps + (size_t)j * C + col + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+            tap[j][e][0] = w4.x; tap[j][e][1] = w4.y; tap[j][e][2] = w4.z; tap[j][e][3] = w4.w;
+        }
+    }
+    const int first = blockIdx.x * run, last = min(first + run, tokens);
+    constexpr int U = 4;    // tokens whose rows and pages are asked for together, before the first of them is used
+    int held = -1;          // the request whose rows the registers hold
+    for (int tu = first; tu < last; tu += U) {
+        float x[U][NV][4];
+        int bs[U], pg[U], at[U];
+#pragma unroll
+        for (int i = 0; i < U; ++i) {
+            const int t = min(tu + i, last - 1);
+            bs[i] = req_of_token[t];
+            at[i] = positions[t];
+#pragma unroll
+            for (int e = 0; e < NV; ++e) {
+                x[i][e][0] = x[i][e][1] = x[i][e][2] = x[i][e][3] = 0.f;
+                if (in[e]) load4<T>(qkv + (size_t)t * row_len + col + lane * 4 + 128 * e, x[i][e]);
+            }
+        }
+#pragma unroll
+        for (int i = 0; i < U; ++i) pg[i] = is_q || bs[i] < 0 ? 0 : block_table[(size_t)bs[i] * table_stride + at[i] / ps];
+#pragma unroll
+        for (int i = 0; i < U; ++i) {
+            const int t = tu + i, b = bs[i];
+            if (t >= last) break;
+            if (b != held) {    // the run's first token, or another request's first token of this step
+                held = b;
+                const int t0 = b >= 0 ? q_start[b] : t, slot = b >= 0 ? slots[b] : -1;
+#pragma unroll
+                for (int j = 0; j < K - 1; ++j) {
+                    const int src = t - (K - 1) + j;
+                    const T* p = src >= t0 ? qkv + (size_t)src * row_len
+                                           : (slot >= 0 ? conv_state + ((size_t)slot * (K - 1) + (K - 1 + src - t0)) * C : nullptr);
+#pragma unroll
+                    for (int e = 0; e < NV; ++e) {
+                        win[j][e][0] = win[j][e][1] = win[j][e][2] = win[j][e][3] = 0.f;
+                        if (p != nullptr && in[e]) load4<T>(p + col + lane * 4 + 128 * e, win[j][e]);
+                    }
+                }
+            }
+            float y[NV][4], ss = 0.f;
+#pragma unroll
+            for (int e = 0; e < NV; ++e)
+#pragma unroll
+                for (int c = 0; c < 4; ++c) {
+                    float v = 0.f;
+#pragma unroll
+                    for (int j = 0; j < K - 1; ++j) v = fmaf(tap[j][e][c], win[j][e][c], v);
+                    v = fmaf(tap[K - 1][e][c], x[i][e][c], v);
+#pragma unroll
+                    for (int j = 0; j + 1 < K - 1; ++j) win[j][e][c] = win[j + 1][e][c];
+                    if (K > 1) win[K - 2 < 0 ? 0 : K - 2][e][c] = x[i][e][c];
+                    y[e][c] = v;
+                    ss = fmaf(v, v, ss);
+                }
+            if (unit) {
+                const float inv = 1.f / sqrtf(warp_sum(ss) / (float)dv + value_eps);
+#pragma unroll
+                for (int e = 0; e < NV; ++e)
+#pragma unroll
+                    for (int c = 0; c < 4; ++c) y[e][c] *= inv;
+            }
+            T* dst;
+            if (is_q) {
+                dst = q_out + ((size_t)t * nh + h) * d;
+            } else {
+                if (b < 0) continue;
+                if (pg[i] < 0 || pg[i] >= num_pages) {
+                    if (lane == 0) atomicOr(err, XB_ERR_BAD_PAGE);
+                    continue;
+                }
+                dst = cache + (((size_t)pg[i] * nkv + g) * ps + at[i] % ps) * len;
+            }
+#pragma unroll
+            for (int e = 0; e < NV; ++e)
+                if (in[e]) store4<T>(dst + lane * 4 + 128 * e, y[e]);
+        }
+    }
+}
+
+template <typename T>
+static bool qkv_conv_runs(T* q_out, T* k_cache, T* v_cache, const T* qkv, long long row_len, const float* taps, int K,
+                          const T* conv_state, const int* positions, const int* req_of_token, const int* block_table,
+                          int table_stride, const int* q_start, const int* slots, int tokens, int nh, int nkv, int d, int dv,
+                          int ps, int num_pages, float value_eps, int write_kv, int* err, cudaStream_t stream) {
+    const int wide = d > dv ? d : dv, heads = nh + 2 * nkv, warps = 8;
+    if (wide > 256 || K > 6) return false;
+    // long enough runs to pay for the K-1 rows read again at a run's start, short enough to fill the machine
+    int run = 32;
+    while (run > 4 && (long long)((tokens + run - 1) / run) * heads < 16 * 148) run /= 2;
+    const dim3 grid((tokens + run - 1) / run, (heads + warps - 1) / warps);
+#define XB_RUNS(KV, NVV)                                                                                                    \
+    qkv_conv_runs_kernel<T, KV, NVV><<<grid, warps * 32, 0, stream>>>(q_out, k_cache, v_cache, qkv, row_len, taps, conv_state, \
+                                                                      positions, req_of_token, block_table, table_stride,   \
+                                                                      q_start, slots, nh, nkv, d, dv, ps, num_pages,        \
+                                                                      value_eps, write_kv, tokens, run, err)
+#define XB_RUNS_K(KV)                                                    \
+    case KV:                                                             \
+        if (wide <= 128) XB_RUNS(KV, 1); else XB_RUNS(KV, 2);            \
+        return true;
+    switch (K) {
+        XB_RUNS_K(1) XB_RUNS_K(2) XB_RUNS_K(3) XB_RUNS_K(4) XB_RUNS_K(5) XB_RUNS_K(6)
+        default: return false;
+    }
+#undef XB_RUNS_K
+#undef XB_RUNS
+}
+
 XB_EXPORT int xb_qkv_prepare(int dtype, void* q_out, void* k_cache, void* v_cache, const void* qkv, const float* q_w,
                              const float* k_w, const float* inv_freq, const int* positions, const int* req_of_token,
                              const int* block_table, int table_stride, int tokens, int nh, int nkv, int d, int dv, int rot,
@@ -399,6 +539,19 @@ XB_EXPORT int xb_qkv_prepare(int dtype, void* q_out, void* k_cache, void* v_cach
     const int vec4 = (d % 4 == 0 && dv % 4 == 0 && row_len % 4 == 0 && v_off % 4 == 0 && (rot % 4 == 0 || value_eps < 0.f) &&
                       !((uintptr_t)taps & 15) && !((uintptr_t)conv_state & (4 * esz - 1)) && !(((uintptr_t)bias | (uintptr_t)q_w | (uintptr_t)k_w) & 15) &&
                       !(((uintptr_t)qkv | (uintptr_t)q_out | (uintptr_t)k_cache | (uintptr_t)v_cache) & (4 * esz - 1))) ? 1 : 0;
+    if (taps && vec4 && tokens > 64 && norm_mode == 0 && !inv_freq && !keep_state && temp_every <= 0) {
+        const bool done =
+            dtype == XB_F32 ? qkv_conv_runs<float>((float*)q_out, (float*)k_cache, (float*)v_cache, (const float*)qkv, row_len, taps,
+                                                   K, (const float*)conv_state, positions, req_of_token, block_table,
+                                                   table_stride, q_start, slots, tokens, nh, nkv, d, dv, page_size, num_pages,
+                                                   value_eps, write_kv, err, stream)
+                            : qkv_conv_runs<__nv_bfloat16>((__nv_bfloat16*)q_out, (__nv_bfloat16*)k_cache, (__nv_bfloat16*)v_cache,
+                                                           (const __nv_bfloat16*)qkv, row_len, taps, K,
+                                                           (const __nv_bfloat16*)conv_state, positions, req_of_token, block_table,
+                                                           table_stride, q_start, slots, tokens, nh, nkv, d, dv, page_size,
+                                                           num_pages, value_eps, write_kv, err, stream);
+        if (done) return xb_launch_status();
+    }
 #define XB_PREPARE(T, CONV)                                                                                               \
     qkv_prepare_kernel<T, CONV><<<dim3(tokens, spread), threads, smem, stream>>>(                                                      \
         (T*)q_out, (T*)k_cache, (T*)v_cache, (const T*)qkv, q_w, k_w, inv_freq, positions, req_of_token, block_table,    \
