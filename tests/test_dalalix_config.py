@@ -155,7 +155,7 @@ def test_blocks_that_disagree_about_the_streams_are_refused():
             BlockSpec("b.", bad).validate()
 
 
-@pytest.mark.parametrize("dims,base", [(24, 10000.0), (6, 40.0), (128, 1e6), (2, 3.0)])
+@pytest.mark.parametrize("dims,base", [(20, 9000.0), (6, 40.0), (128, 1e6), (2, 3.0)])
 def test_frequencies_of_the_product_equal_the_plain_ones(dims, base):
     want = torch.tensor([base ** (-2.0 * i / dims) for i in range(dims // 2)], dtype=F64)
     got = torch.from_numpy(inv_frequencies(base, dims, None, True)).double()

@@ -88,8 +88,10 @@ __device__ __forceinline__ PrefillItem prefill_item(const int* __restrict__ item
 
 // `work`: [ctas + 1] offsets into the items that follow them, PREFILL_ITEM_INTS int32 each; CTA c takes
 // items work[c] .. work[c + 1] - 1 in that order.
-template <int DP>
-__global__ void __launch_bounds__(PREFILL_THREADS)
+// EXT false: the attention without a cap, a bias on the distance, kept first positions, a sink or an output scale, compiled
+// without the code for them.
+template <int DP, bool EXT>
+__global__ void __launch_bounds__(PREFILL_THREADS, DP == 64 ? 1 : 0)   // (the hint measured better at 64 channels, worse at 128)
 attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                        const __grid_constant__ CUtensorMap map_v, const __grid_constant__ CUtensorMap map_o,
                        __nv_bfloat16* __restrict__ out, const int* __restrict__ q_start, const int* __restrict__ start_pos,
@@ -97,6 +99,12 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
                        int ps, int ps_shift, int num_pages, int window, int keep, float scale_log2_in, float softcap,
                        float slope_exp, const float* __restrict__ sink, float out_scale,
                        const int* __restrict__ work, int* err) {
+    if (!EXT) {
+        softcap = slope_exp = 0.f;
+        keep = 0;
+        sink = nullptr;
+        out_scale = 1.f;
+    }
     // changed scores (a cap, a bias on the distance): the scores are brought to their final values first and the
     // softmax then only changes the base of the exponential
     const bool changed = softcap > 0.f || slope_exp > 0.f;
@@ -686,8 +694,8 @@ attn_decode_plan_kernel(int* __restrict__ plan, int capacity, const int* __restr
 // when a row's reference maximum has to move (then O is rescaled in TMEM).  The pieces of one token
 // and head are merged by the CTA that finishes last (a ticket per token and key/value head), in
 // the order of the pieces.
-template <int DP>
-__global__ void __launch_bounds__(128)
+template <int DP, bool EXT>
+__global__ void __launch_bounds__(128, 2)
 attn_decode_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                       const __grid_constant__ CUtensorMap map_v, __nv_bfloat16* __restrict__ out,
                       float* __restrict__ part_o, float* __restrict__ part_ml, const int* __restrict__ plan,
@@ -696,6 +704,12 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
                       const float* __restrict__ sink, float out_scale, int dec_max,
                       int splits_max, int page_cap, int* __restrict__ tickets, int* err) {
     constexpr int HALVES = DP / 64, DEC_STAGES = dec_stages(DP);
+    if (!EXT) {     // as for the prefill kernel
+        softcap = slope_exp = 0.f;
+        keep = 0;
+        sink = nullptr;
+        out_scale = 1.f;
+    }
     // changed scores (a cap, a bias on the distance): brought to their final values before the softmax, which then
     // only changes the base of the exponential
     const bool changed = softcap > 0.f || slope_exp > 0.f;
@@ -1129,6 +1143,11 @@ bool map_q3(CUtensorMap* out, const void* ptr, long long T, int nh, int d, long 
     return tensor_map_bf16(out, ptr, 3, dims, strides, box);
 }
 
+// whether a launch needs the kernels' code for anything but the plain attention
+bool changed_attention(float softcap, float slope_exp, int keep, const float* sink, float out_scale) {
+    return softcap > 0.f || slope_exp > 0.f || keep > 0 || sink != nullptr || out_scale != 1.f;
+}
+
 template <int DP>
 int launch_prefill(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, const CUtensorMap& mo, void* out,
                    const int* q_start, const int* start_pos, const int* table, int stride, int nh, int nkv, int dv,
@@ -1138,9 +1157,11 @@ int launch_prefill(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorM
     // Q of two heads, the key/value stages, the barriers' kilobyte, 4 KB of output staging per softmax warp and half
     constexpr size_t smem = 2 * (size_t)(DP / 64) * QT * 128 + PREFILL_STAGES * 2 * (size_t)(DP / 64) * KT * 128 + 1024 +
                             8 * (size_t)(DP / 64) * 4096;
-    cudaFuncSetAttribute(attn_prefill_tc_kernel<DP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    cudaFuncSetAttribute(attn_prefill_tc_kernel<DP>, cudaFuncAttributePreferredSharedMemoryCarveout, 100);
-    return xb_launch(attn_prefill_tc_kernel<DP>, dim3(ctas), dim3(PREFILL_THREADS), smem, stream, mq, mk, mv, mo,
+    const auto kernel = changed_attention(softcap, slope_exp, keep, sink, out_scale) ? attn_prefill_tc_kernel<DP, true>
+                                                                                    : attn_prefill_tc_kernel<DP, false>;
+    cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    cudaFuncSetAttribute(kernel, cudaFuncAttributePreferredSharedMemoryCarveout, 100);
+    return xb_launch(kernel, dim3(ctas), dim3(PREFILL_THREADS), smem, stream, mq, mk, mv, mo,
                      (__nv_bfloat16*)out, q_start, start_pos, table, stride, nh, nkv, dv, ldo, ps, ps_shift, num_pages,
                      window, keep, sl2, softcap, slope_exp, sink, out_scale, work, err);
 }
@@ -1155,9 +1176,11 @@ int launch_decode(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMa
                   cudaStream_t stream) {
     constexpr size_t smem = (size_t)(DP / 64) * DEC_ROWS * 128 + 2 * DEC_ROWS * 128 + dec_stages(DP) * 2 * (size_t)(DP / 64) * KT * 128 +
                             32 * dec_stages(DP) + 96 + (size_t)DEC_PAGE_CAP * 4;
-    cudaFuncSetAttribute(attn_decode_tc_kernel<DP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    cudaFuncSetAttribute(attn_decode_tc_kernel<DP>, cudaFuncAttributePreferredSharedMemoryCarveout, 100);
-    return xb_launch_opt(overlap != 0, attn_decode_tc_kernel<DP>, dim3(nkv, pieces), dim3(128), smem, stream, mq, mk, mv,
+    const auto kernel = changed_attention(softcap, slope_exp, keep, sink, out_scale) ? attn_decode_tc_kernel<DP, true>
+                                                                                    : attn_decode_tc_kernel<DP, false>;
+    cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    cudaFuncSetAttribute(kernel, cudaFuncAttributePreferredSharedMemoryCarveout, 100);
+    return xb_launch_opt(overlap != 0, kernel, dim3(nkv, pieces), dim3(128), smem, stream, mq, mk, mv,
                          (__nv_bfloat16*)out, part_o, part_ml, plan, table, stride, nh, nkv, dv, ldo, ps, ps_shift, num_pages,
                          keep, sl2, softcap, slope_exp, sink, out_scale, dec_max, splits_max, DEC_PAGE_CAP, tickets, err);
 }
